@@ -4,6 +4,7 @@ from .zatupel import ZatupelConfig
 from .tidenex import TidenexConfig
 from .tuzavik import TuzavikConfig
 from .natalorn import NatalornConfig
+from .ramupel import RamupelConfig
 from .registry import (config_from_dict, load_config, register_architecture, registered_architectures,
                        unregister_architecture)
 
@@ -26,5 +27,9 @@ register_architecture("Tuzavik", TuzavikConfig, replace=True)
 # attention over one cached latent per token with a sink and a gate, routed experts chosen within groups beside a shared expert
 register_architecture("Natalorn", NatalornConfig, replace=True)
 
-__all__ = ["ZatupelConfig", "TidenexConfig", "TuzavikConfig", "NatalornConfig", "ConfigError", "LayerSpec", "ModelPlan", "PartSpec", "LlamaConfig", "config_from_dict", "load_config",
+# parallel layers with a gate per channel on every sublayer's result, and a stream that is averaged over the depth: attention over
+# one cached latent per token with a gate per head, or gated linear attention; ungated feed-forwards
+register_architecture("Ramupel", RamupelConfig, replace=True)
+
+__all__ = ["ZatupelConfig", "TidenexConfig", "TuzavikConfig", "NatalornConfig", "RamupelConfig", "ConfigError", "LayerSpec", "ModelPlan", "PartSpec", "LlamaConfig", "config_from_dict", "load_config",
            "register_architecture", "registered_architectures", "unregister_architecture"]

@@ -55,6 +55,9 @@ class ModelPlan:
     # the residual stream is kept as this many copies (all equal to the embedding output at the start; the final norm reads their
     # sum); the layers' blocks then work on rows of streams * hidden_size numbers
     streams: int = 1
+    # what every layer leaves is kept, and the layers' blocks work on the whole history, planes [runs + 1, T, hidden_size] (the
+    # embedding output first, the stream last)
+    depth_average: bool = False
 
 
 def require(d, key, typ):

@@ -13,7 +13,8 @@
 //                      input channels that are rotated and copied behind the N outputs (the absorbed query)
 //   latent_attention   causal softmax attention over the latent rows, fp32 arithmetic whatever the storage type
 //
-// The rotation pairs channel 2i with 2i + 1 and turns the pair by position * freq[i]; cos and sin are multiplied by `amp`.
+// The rotation pairs channel 2i with 2i + 1, or (halves) channel i with i + R/2, and turns the pair by position * freq[i]; cos and
+// sin are multiplied by `amp`.
 // Keys are walked in chunks of KT positions that start at multiples of KT, a chunk's weights are summed in a fixed order,
 // and a key that a token does not see adds exact zeros: what a token adds up, and in which order, depends on its position
 // alone, not on the step's cut, the tile, or the batch around it.
@@ -25,22 +26,29 @@ namespace {
 
 constexpr int kPrepThreads = 128;
 
-// One CTA per token.  proj fp32 row = [dq: Cq | c: C | kr: R] (C = 0: a layer that reads another layer's rows and has only dq).
+// Where the two channels of rotated pair i lie among R channels.
+__device__ __forceinline__ int pair_first(int i, int halves) { return halves ? i : 2 * i; }
+__device__ __forceinline__ int pair_second(int i, int R, int halves) { return halves ? i + (R >> 1) : 2 * i + 1; }
+
+// One CTA per token.  proj fp32 row = [dq: Cq | c: C | kr: R] (C = 0: a layer that reads another layer's rows and has only dq;
+// Cq = 0: a layer whose queries do not come from a latent).
 template <typename TC>
 __global__ void __launch_bounds__(kPrepThreads)
 latent_prepare_kernel(const float* __restrict__ proj, int ld, const int32_t* __restrict__ positions,
                       const int32_t* __restrict__ slot_mapping, const float* __restrict__ freq, float amp,
                       const float* __restrict__ wq, const float* __restrict__ wc, TC* __restrict__ cq_out, TC* __restrict__ cache,
-                      int Cq, int C, int R, float eps) {
+                      int Cq, int C, int R, float eps, int halves) {
     __shared__ float red[32];
     forge::pdl_launch_dependents();
     forge::pdl_wait();
     const int t = blockIdx.x;
     const float* row = proj + (size_t)t * ld;
     float ss = 0.f;
-    for (int i = threadIdx.x; i < Cq; i += kPrepThreads) ss = fmaf(row[i], row[i], ss);
-    const float inv_q = 1.0f / sqrtf(forge::block_sum(ss, red) / (float)Cq + eps);
-    for (int i = threadIdx.x; i < Cq; i += kPrepThreads) cq_out[(size_t)t * Cq + i] = forge::from_float<TC>(row[i] * inv_q * wq[i]);
+    if (Cq > 0) {
+        for (int i = threadIdx.x; i < Cq; i += kPrepThreads) ss = fmaf(row[i], row[i], ss);
+        const float inv_q = 1.0f / sqrtf(forge::block_sum(ss, red) / (float)Cq + eps);
+        for (int i = threadIdx.x; i < Cq; i += kPrepThreads) cq_out[(size_t)t * Cq + i] = forge::from_float<TC>(row[i] * inv_q * wq[i]);
+    }
     if (C == 0 || slot_mapping == nullptr) return;
     const int slot = slot_mapping[t];
     if (slot < 0 || !FORGE_SLOT_OK(slot)) return;
@@ -56,9 +64,10 @@ latent_prepare_kernel(const float* __restrict__ proj, int ld, const int32_t* __r
         sincosf(pos * freq[i], &sn, &cs);
         sn *= amp;
         cs *= amp;
-        const float u = c[C + 2 * i], v = c[C + 2 * i + 1];
-        dst[C + 2 * i] = forge::from_float<TC>(u * cs - v * sn);
-        dst[C + 2 * i + 1] = forge::from_float<TC>(v * cs + u * sn);
+        const int a = C + pair_first(i, halves), b = C + pair_second(i, R, halves);
+        const float u = c[a], v = c[b];
+        dst[a] = forge::from_float<TC>(u * cs - v * sn);
+        dst[b] = forge::from_float<TC>(v * cs + u * sn);
     }
 }
 
@@ -70,7 +79,7 @@ template <typename TI, typename TW, typename TO>
 __global__ void __launch_bounds__(kLinThreads)
 head_linear_kernel(const TI* __restrict__ in, long long in_ld, int in_hs, const TW* __restrict__ W, TO* __restrict__ out,
                    long long out_ld, int out_hs, const int32_t* __restrict__ positions, const float* __restrict__ freq, float amp,
-                   int T, int K, int N, int R, const float* __restrict__ gate, long long gate_ld) {
+                   int T, int K, int N, int R, const float* __restrict__ gate, long long gate_ld, int gate_hs, int gate_cs, int halves) {
     extern __shared__ float xs[];                       // [kLinTokens][K]
     forge::pdl_launch_dependents();
     forge::pdl_wait();
@@ -95,7 +104,7 @@ head_linear_kernel(const TI* __restrict__ in, long long in_ld, int in_hs, const 
         for (int tt = 0; tt < kLinTokens; ++tt)
             if (tt < nt) {
                 float v = acc[tt];
-                if (gate) v *= 1.0f / (1.0f + expf(-gate[(size_t)(t0 + tt) * gate_ld + (size_t)h * N + n]));
+                if (gate) v *= 1.0f / (1.0f + expf(-gate[(size_t)(t0 + tt) * gate_ld + (size_t)h * gate_hs + n * gate_cs]));
                 out[(size_t)(t0 + tt) * out_ld + (size_t)h * out_hs + n] = forge::from_float<TO>(v);
             }
     }
@@ -107,10 +116,11 @@ head_linear_kernel(const TI* __restrict__ in, long long in_ld, int in_hs, const 
             sincosf((float)positions[t0 + tt] * freq[p], &sn, &cs);
             sn *= amp;
             cs *= amp;
-            const float u = forge::to_float(src[2 * p]), v = forge::to_float(src[2 * p + 1]);
+            const int a = pair_first(p, halves), b = pair_second(p, R, halves);
+            const float u = forge::to_float(src[a]), v = forge::to_float(src[b]);
             TO* dst = out + (size_t)(t0 + tt) * out_ld + (size_t)h * out_hs + N;
-            dst[2 * p] = forge::from_float<TO>(u * cs - v * sn);
-            dst[2 * p + 1] = forge::from_float<TO>(v * cs + u * sn);
+            dst[a] = forge::from_float<TO>(u * cs - v * sn);
+            dst[b] = forge::from_float<TO>(v * cs + u * sn);
         }
     }
 }
@@ -149,7 +159,7 @@ template <typename TI>
 __global__ void __launch_bounds__(kHlmThreads)
 head_linear_mma_kernel(const TI* __restrict__ in, long long in_ld, int in_hs, const __nv_bfloat16* __restrict__ W, __nv_bfloat16* __restrict__ out,
                        long long out_ld, int out_hs, const int32_t* __restrict__ positions, const float* __restrict__ freq, float amp,
-                       int T, int K, int N, int R, const float* __restrict__ gate, long long gate_ld) {
+                       int T, int K, int N, int R, const float* __restrict__ gate, long long gate_ld, int gate_hs, int gate_cs, int halves) {
     __shared__ __align__(16) __nv_bfloat16 As[kHlmTile][kHlmRowK];         // [token][input channel of the chunk]
     __shared__ __align__(16) __nv_bfloat16 Bs[kHlmK][kHlmRow];             // [input channel of the chunk][output channel]
     forge::pdl_launch_dependents();
@@ -214,9 +224,9 @@ head_linear_mma_kernel(const TI* __restrict__ in, long long in_ld, int in_hs, co
             __nv_bfloat16* dst = out + (size_t)t * out_ld + (size_t)h * out_hs + n;
             float v0 = acc[nb][2 * half], v1 = acc[nb][2 * half + 1];
             if (gate) {
-                const float* gr = gate + (size_t)t * gate_ld + (size_t)h * N + n;
-                if (n < N) v0 *= 1.0f / (1.0f + expf(-gr[0]));
-                if (n + 1 < N) v1 *= 1.0f / (1.0f + expf(-gr[1]));
+                const float* gr = gate + (size_t)t * gate_ld + (size_t)h * gate_hs;
+                if (n < N) v0 *= 1.0f / (1.0f + expf(-gr[n * gate_cs]));
+                if (n + 1 < N) v1 *= 1.0f / (1.0f + expf(-gr[(n + 1) * gate_cs]));
             }
             if (n < N) dst[0] = __float2bfloat16(v0);
             if (n + 1 < N) dst[1] = __float2bfloat16(v1);
@@ -230,10 +240,11 @@ head_linear_mma_kernel(const TI* __restrict__ in, long long in_ld, int in_hs, co
             sincosf((float)positions[t0 + tt] * freq[p], &sn, &cs);
             sn *= amp;
             cs *= amp;
-            const float u = forge::to_float(src[2 * p]), v = forge::to_float(src[2 * p + 1]);
+            const int a = pair_first(p, halves), b = pair_second(p, R, halves);
+            const float u = forge::to_float(src[a]), v = forge::to_float(src[b]);
             __nv_bfloat16* dst = out + (size_t)(t0 + tt) * out_ld + (size_t)h * out_hs + N;
-            dst[2 * p] = __float2bfloat16(u * cs - v * sn);
-            dst[2 * p + 1] = __float2bfloat16(v * cs + u * sn);
+            dst[a] = __float2bfloat16(u * cs - v * sn);
+            dst[b] = __float2bfloat16(v * cs + u * sn);
         }
     }
 }
@@ -353,38 +364,41 @@ forge::PerDeviceFlag g_latent_attr[2];
 template <typename TI, typename TW, typename TO>
 cudaError_t launch_head_linear(cudaStream_t stream, const void* in, long long in_ld, int in_hs, const void* W, void* out, long long out_ld,
                                int out_hs, const int32_t* positions, const float* freq, float amp, int T, int H, int K, int N, int R, const float* gate,
-                               long long gate_ld) {
+                               long long gate_ld, int gate_hs, int gate_cs, int halves) {
     const dim3 grid((T + kLinTokens - 1) / kLinTokens, H, (N + kLinThreads - 1) / kLinThreads);
     return forge::launch(head_linear_kernel<TI, TW, TO>, grid, dim3(kLinThreads), sizeof(float) * kLinTokens * K, stream, 1, (const TI*)in,
-                         in_ld, in_hs, (const TW*)W, (TO*)out, out_ld, out_hs, positions, freq, amp, T, K, N, R, gate, gate_ld);
+                         in_ld, in_hs, (const TW*)W, (TO*)out, out_ld, out_hs, positions, freq, amp, T, K, N, R, gate, gate_ld, gate_hs,
+                         gate_cs, halves);
 }
 
 }  // namespace
 
-// proj fp32 [T, ld]: Cq channels of the query's down-projection, then (C > 0) C + R of the key/value one.  wq fp32 [Cq],
+// proj fp32 [T, ld]: Cq channels of the query's down-projection (0: none), then (C > 0) C + R of the key/value one.  wq fp32 [Cq],
 // wc fp32 [C]; freq fp32 [R/2].  cq_out [T, Cq] and cache (rows of C + R, row = slot) of type dtype.  slot_mapping null
-// or C = 0: nothing stored.
+// or C = 0: nothing stored.  halves: the rotation pairs channel i with i + R/2 (0: 2i with 2i + 1).
 extern "C" int forge_latent_prepare(const float* proj, int ld, const int32_t* positions, const int32_t* slot_mapping, const float* freq,
                                     float amp, const float* wq, const float* wc, void* cq_out, void* cache, int dtype, int T, int Cq,
-                                    int C, int R, float eps, cudaStream_t stream) {
-    if (T < 0 || Cq <= 0 || C < 0 || R < 0 || (R & 1) || ld < Cq + (C > 0 ? C + R : 0))
+                                    int C, int R, float eps, int halves, cudaStream_t stream) {
+    if (T < 0 || Cq < 0 || (Cq > 0 && (!wq || !cq_out)) || (Cq == 0 && C <= 0) || C < 0 || R < 0 || (R & 1) || ld < Cq + (C > 0 ? C + R : 0))
         return forge::fail(FORGE_ERR_ARG, "latent_prepare: bad sizes T=%d Cq=%d C=%d R=%d ld=%d", T, Cq, C, R, ld);
     if (C > 0 && slot_mapping && (!cache || !wc || (R > 0 && !freq))) return forge::fail(FORGE_ERR_ARG, "latent_prepare: the cache write needs its tensors");
     if (T == 0) return FORGE_OK;
     cudaError_t e = cudaSuccess;
     FORGE_DISPATCH_DTYPE(dtype, TT,
         e = forge::launch(latent_prepare_kernel<TT>, dim3(T), dim3(kPrepThreads), 0, stream, 1, proj, ld, positions, slot_mapping, freq, amp, wq,
-                          wc, (TT*)cq_out, (TT*)cache, Cq, C, R, eps));
+                          wc, (TT*)cq_out, (TT*)cache, Cq, C, R, eps, halves));
     return forge::check_launch("latent_prepare", e);
 }
 
 // out[t, h, 0:N] = sum_k in[t, h, k] W[h, k, n], and (R > 0) out[t, h, N:N+R] = in[t, h, K:K+R] rotated by positions[t].
 // in of in_dtype (fp32 or bf16), W and out of dtype; leading dimensions and head strides in elements.  bf16 weights go to the
 // tensor cores (fp32 inputs rounded to bfloat16 on the way) unless `simt` asks for the fp32 multiply-adds.  gate fp32 (rows of
-// gate_ld, head h's N numbers from h * N) or null: out[t, h, n] is multiplied by sigmoid(gate[t, h, n]).
+// gate_ld) or null: out[t, h, n] is multiplied by sigmoid(gate[t][h * gate_hs + n * gate_cs]) (a gate per channel: N and 1; one per
+// head: 1 and 0).  halves: the rotation pairs channel i with i + R/2 (0: 2i with 2i + 1).
 extern "C" int forge_head_linear(const void* in, int in_dtype, long long in_ld, int in_hs, const void* W, void* out, int dtype,
                                  long long out_ld, int out_hs, const int32_t* positions, const float* freq, float amp, int T, int H,
-                                 int K, int N, int R, int simt, const float* gate, long long gate_ld, cudaStream_t stream) {
+                                 int K, int N, int R, int simt, const float* gate, long long gate_ld, int gate_hs, int gate_cs, int halves,
+                                 cudaStream_t stream) {
     if (T < 0 || H <= 0 || K <= 0 || N <= 0 || R < 0 || (R & 1)) return forge::fail(FORGE_ERR_ARG, "head_linear: bad sizes T=%d H=%d K=%d N=%d R=%d", T, H, K, N, R);
     if (R > 0 && (!positions || !freq)) return forge::fail(FORGE_ERR_ARG, "head_linear: a rotation needs positions and frequencies");
     if (T == 0) return FORGE_OK;
@@ -393,19 +407,21 @@ extern "C" int forge_head_linear(const void* in, int in_dtype, long long in_ld, 
         const dim3 grid((T + kHlmTile - 1) / kHlmTile, H, (N + kHlmTile - 1) / kHlmTile);
         if (in_dtype == FORGE_F32)
             e = forge::launch(head_linear_mma_kernel<float>, grid, dim3(kHlmThreads), 0, stream, 1, (const float*)in, in_ld, in_hs,
-                              (const __nv_bfloat16*)W, (__nv_bfloat16*)out, out_ld, out_hs, positions, freq, amp, T, K, N, R, gate, gate_ld);
+                              (const __nv_bfloat16*)W, (__nv_bfloat16*)out, out_ld, out_hs, positions, freq, amp, T, K, N, R, gate, gate_ld, gate_hs,
+                              gate_cs, halves);
         else
             e = forge::launch(head_linear_mma_kernel<__nv_bfloat16>, grid, dim3(kHlmThreads), 0, stream, 1, (const __nv_bfloat16*)in, in_ld, in_hs,
-                              (const __nv_bfloat16*)W, (__nv_bfloat16*)out, out_ld, out_hs, positions, freq, amp, T, K, N, R, gate, gate_ld);
+                              (const __nv_bfloat16*)W, (__nv_bfloat16*)out, out_ld, out_hs, positions, freq, amp, T, K, N, R, gate, gate_ld, gate_hs,
+                              gate_cs, halves);
         return forge::check_launch("head_linear (tensor cores)", e);
     }
     if (sizeof(float) * kLinTokens * K > 48 * 1024) return forge::fail(FORGE_ERR_UNSUPPORTED, "head_linear: %d input channels a head", K);
     if (dtype == FORGE_F32 && in_dtype == FORGE_F32)
-        e = launch_head_linear<float, float, float>(stream, in, in_ld, in_hs, W, out, out_ld, out_hs, positions, freq, amp, T, H, K, N, R, gate, gate_ld);
+        e = launch_head_linear<float, float, float>(stream, in, in_ld, in_hs, W, out, out_ld, out_hs, positions, freq, amp, T, H, K, N, R, gate, gate_ld, gate_hs, gate_cs, halves);
     else if (dtype == FORGE_BF16 && in_dtype == FORGE_F32)
-        e = launch_head_linear<float, __nv_bfloat16, __nv_bfloat16>(stream, in, in_ld, in_hs, W, out, out_ld, out_hs, positions, freq, amp, T, H, K, N, R, gate, gate_ld);
+        e = launch_head_linear<float, __nv_bfloat16, __nv_bfloat16>(stream, in, in_ld, in_hs, W, out, out_ld, out_hs, positions, freq, amp, T, H, K, N, R, gate, gate_ld, gate_hs, gate_cs, halves);
     else if (dtype == FORGE_BF16 && in_dtype == FORGE_BF16)
-        e = launch_head_linear<__nv_bfloat16, __nv_bfloat16, __nv_bfloat16>(stream, in, in_ld, in_hs, W, out, out_ld, out_hs, positions, freq, amp, T, H, K, N, R, gate, gate_ld);
+        e = launch_head_linear<__nv_bfloat16, __nv_bfloat16, __nv_bfloat16>(stream, in, in_ld, in_hs, W, out, out_ld, out_hs, positions, freq, amp, T, H, K, N, R, gate, gate_ld, gate_hs, gate_cs, halves);
     else
         return forge::fail(FORGE_ERR_ARG, "head_linear: input type %d with weights of type %d", in_dtype, dtype);
     return forge::check_launch("head_linear", e);

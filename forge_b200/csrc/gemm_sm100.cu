@@ -51,6 +51,7 @@ struct GemmParams {
     int NH, NKV, head_dim, page_size;
     // a device word that an earlier kernel wrote: where it holds 0 the whole product is skipped (nothing is read or written); null: none
     const int* live;
+    float act_a, act_b;              // numbers of the activation in the bfloat16 store (builds with -DFORGE_CAST_ACT=2)
 };
 
 // Every thread of every CTA leaves before anything is set up (no barrier, tensor memory or copy exists yet), all the same way.
@@ -78,13 +79,19 @@ template <int BN> struct Cfg {
 #define FORGE_GATE_GELU 0
 #endif
 // The activation of the epilogue that stores bfloat16 (EPI_STORE_BF16): none in the ordinary build; in a library built with
-// -DFORGE_CAST_ACT=1 the exact gelu, v/2 (1 + erf(v / sqrt 2)), the activation between the two products of an ungated
-// feed-forward.  A variant of its own for the same reason as the gelu gate: the ordinary build's epilogues stay as they were.
+// -DFORGE_CAST_ACT=1 the exact gelu, v/2 (1 + erf(v / sqrt 2)), with -DFORGE_CAST_ACT=2 xIELU with the call's two curvatures
+// (a v^2 + v/2 above zero, b (exp(v) - 1 - v) + v/2 below): activations between the two products of an ungated feed-forward.
+// The difference exp(v) - 1 - v loses digits near zero, where it is b times some 1e-7 beside v/2, far below the store's rounding.  A variant of its own for the same reason as the gelu gate: the ordinary build's epilogues stay as they were.
 #ifndef FORGE_CAST_ACT
 #define FORGE_CAST_ACT 0
 #endif
 #if FORGE_CAST_ACT == 1
 #define FORGE_CAST(v) (0.5f * (v) * (1.0f + erff((v) * 0.7071067811865476f)))
+#elif FORGE_CAST_ACT == 2
+#define FORGE_CAST(v) xielu((v), p.act_a, p.act_b)
+__device__ __forceinline__ float xielu(float v, float a, float b) {
+    return fmaf(0.5f, v, v > 0.f ? a * v * v : b * (__expf(v) - 1.0f - v));
+}
 #else
 #define FORGE_CAST(v) (v)
 #endif
@@ -1778,7 +1785,7 @@ extern "C" int forge_gemm_sm100_set_workspace(void* ptr, long long bytes) {
 // the few-rows kernel with K cut across a cluster of that many CTAs; -100 (M <= 64 only) = the few-rows kernel
 // that deals units of work out evenly to persistent CTAs (the default once a workspace has been set).  status: device int, bit 1 raised if a wait ran out.
 extern "C" int forge_gemm_sm100(const void* A, const void* W, const float* bias, void* C, int* status, int M, int N,
-                                int K, int epilogue, int tile_n, const int* live, cudaStream_t stream) {
+                                int K, int epilogue, int tile_n, const int* live, float act_a, float act_b, cudaStream_t stream) {
     if (M < 0 || N <= 0 || K <= 0) return forge::fail(FORGE_ERR_ARG, "gemm_sm100: bad sizes M=%d N=%d K=%d", M, N, K);
     if (M == 0) return FORGE_OK;
     if (K % 8 != 0) return forge::fail(FORGE_ERR_UNSUPPORTED, "gemm_sm100: K=%d is not a multiple of 8 (TMA row stride)", K);
@@ -1813,7 +1820,7 @@ extern "C" int forge_gemm_sm100(const void* A, const void* W, const float* bias,
             if (!bf16_tile_map(W, N, K, BM, &tw, &err)) return forge::fail(FORGE_ERR_UNSUPPORTED, "gemm_sm100: W: %s", err);
             if (!bf16_tile_map(A, M, K, nt, &tx, &err)) return forge::fail(FORGE_ERR_UNSUPPORTED, "gemm_sm100: A: %s", err);
             GemmParams p{C, bias, M, N, K, epilogue, status};
-            p.live = live;
+            p.live = live; p.act_a = act_a; p.act_b = act_b;
             switch (nt) {
                 case 16: return launch_streamk<16>(tw, tx, p, stream);
                 case 32: return launch_streamk<32>(tw, tx, p, stream);
@@ -1865,7 +1872,7 @@ extern "C" int forge_gemm_sm100(const void* A, const void* W, const float* bias,
         // 128-wide tiles is the faster one there (22 against 28-33 us at [11264 x 2048])
         const bool token_major_instead = nt == 128 && tile_n == 0 && ksplit == 1;
         GemmParams p{C, bias, M, N, K, epilogue, status};
-        p.live = live;
+        p.live = live; p.act_a = act_a; p.act_b = act_b;
         if (!token_major_instead) switch (nt) {
             case 16: return launch_skinny<16>(W, A, p, ksplit, tile_rows, stream);
             case 32: return launch_skinny<32>(W, A, p, ksplit, tile_rows, stream);
@@ -1888,7 +1895,7 @@ extern "C" int forge_gemm_sm100(const void* A, const void* W, const float* bias,
         }
         if (ks > 0) {
             GemmParams p{C, bias, M, N, K, epilogue, status};
-            p.live = live;
+            p.live = live; p.act_a = act_a; p.act_b = act_b;
             return launch_splitk(A, W, p, ks, stream);
         }
     }
@@ -1925,7 +1932,7 @@ extern "C" int forge_gemm_sm100(const void* A, const void* W, const float* bias,
     if (bn == 512 || bn == 1192 || bn == 1128) {
         if (M <= BM) return forge::fail(FORGE_ERR_ARG, "gemm_sm100: the two-CTA tile is for more than %d rows, got %d", BM, M);
         GemmParams p{C, bias, M, N, K, epilogue, status};
-        p.live = live;
+        p.live = live; p.act_a = act_a; p.act_b = act_b;
         if (bn == 512) return launch_pair(A, W, p, stream);
         if (K % BK != 0 || K < 2 * BK)
             return forge::fail(FORGE_ERR_UNSUPPORTED, "gemm_sm100: two-CTA tiles of %d columns need K %% 64 == 0 and K >= 128, got %d", bn - 1000, K);
@@ -1935,7 +1942,7 @@ extern "C" int forge_gemm_sm100(const void* A, const void* W, const float* bias,
     if (!bf16_tile_map(A, M, K, BM, &ta, &err)) return forge::fail(FORGE_ERR_UNSUPPORTED, "gemm_sm100: A: %s", err);
     if (!bf16_tile_map(W, N, K, bn, &tw, &err)) return forge::fail(FORGE_ERR_UNSUPPORTED, "gemm_sm100: W: %s", err);
     GemmParams p{C, bias, M, N, K, epilogue, status};
-    p.live = live;
+    p.live = live; p.act_a = act_a; p.act_b = act_b;
     switch (bn) {
         case 256: return launch<256>(ta, tw, p, stream);
         case 224: return launch<224>(ta, tw, p, stream);

@@ -126,7 +126,7 @@ rmsnorm_pair_kernel(const float* __restrict__ x, const float* __restrict__ w1, c
     }
 }
 
-// Layer norm with weight and bias:  y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b.  One CTA per row; the mean
+// Layer norm with a weight and (b not null) a bias:  y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b.  One CTA per row; the mean
 // first, then the mean of the squared deviations from it (not E[x^2] - mean^2), both with the fixed reduction tree.
 template <typename TOut>
 __global__ void __launch_bounds__(kNormThreads)
@@ -147,7 +147,7 @@ layernorm_kernel(const float* __restrict__ x, const float* __restrict__ w, const
         ss = fmaf(d, d, ss);
     }
     const float inv = 1.0f / sqrtf(forge::block_sum(ss, red) / (float)H + eps);
-    for (int c = threadIdx.x; c < H; c += kNormThreads) o[c] = forge::from_float<TOut>(fmaf((xr[c] - mean) * inv, w[c], b[c]));
+    for (int c = threadIdx.x; c < H; c += kNormThreads) o[c] = forge::from_float<TOut>(fmaf((xr[c] - mean) * inv, w[c], b ? b[c] : 0.f));
 }
 
 // A sublayer's output y joins the stream through a norm of its own:  r <- r + mult * y / rms(y) * w_y, and, where the next

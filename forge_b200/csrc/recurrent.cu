@@ -13,7 +13,10 @@
 //   retention:                 S <- g S + k_t v_t^T ;   o_t = S^T q_t                         (one fixed decay g per head; q and k
 //                              rotated by their position, k times K^-1/2, by retention_prepare_kernel)
 //
-// In the last two the state is [K, V] with V value channels that need not equal K; the first two have V = K.
+//   gated linear attention:    S <- diag(a_t) S + k_t v_t^T ;   o_t = K^-1/2 S^T q_t            (a decay per key channel from a
+//                              a_t = sigmoid(W2 u_t + b)^(1/tau)                                 low-rank projection, lowrank_decay_kernel)
+//
+// In the last three the state is [K, V] with V value channels that need not equal K; the first two have V = K.
 //
 // A CTA per (request, head, 16 columns of S) walks the request's tokens of the step in order; column j of S (the K numbers
 // that meet value channel j) lives in the registers of eight neighbouring threads, so a token costs K/8 multiply-adds per
@@ -24,7 +27,7 @@
 
 namespace {
 
-constexpr int kScanTokens = 8;        // tokens whose vectors are staged at a time
+constexpr int kScanTokens = 8;        // tokens whose vectors are staged at a time (at most)
 
 struct ScanInput {                    // a [T, heads * K] fp32 matrix that may be a column slice of a wider one
     const float* p;
@@ -86,7 +89,8 @@ __device__ __forceinline__ void stage_async(float* dst, const float* src, int by
 }
 
 // MODE 0: decay and bonus; MODE 1: generalized delta rule; MODE 2: gated write (no k: 1 - d stands for it; KV value
-// channels, the columns of S).  d: the decays, a: the removal rates (MODE 1), both ready made
+// channels, the columns of S); MODE 3: retention (one decay per head); MODE 4: gated linear attention (KV value channels; what
+// comes out is multiplied by out_scale).  d: the decays, a: the removal rates (MODE 1), both ready made
 // (scan_gates_kernel).  last_in (MODE 0, may be null): the mixer's input rows [T, W] of the activation type; the
 // request's last row is kept as fp32 at state + prev_off (the next step's "previous token").
 //
@@ -101,8 +105,9 @@ __global__ void __launch_bounds__(kScanThreads)
 state_scan_kernel(ScanInput r, ScanInput k, ScanInput v, ScanInput d, ScanInput a, const float* __restrict__ bonus,
                   const float* __restrict__ inv, float* __restrict__ state, long long state_stride, const int32_t* __restrict__ q_start,
                   const int32_t* __restrict__ slots, float* __restrict__ out, const TA* __restrict__ last_in, int W,
-                  long long prev_off, int N, int K, int KV, int vec) {
+                  long long prev_off, int N, int K, int KV, int vec, float out_scale) {
     constexpr int RPT = KMAX / kSplit;                                  // rows of S per thread
+    constexpr int kScanTokens = MODE == 4 && KMAX > 192 ? 4 : ::kScanTokens;   // (three vectors of 256 channels: four tokens fit 48 KB)
     __shared__ __align__(16) float rs[2][kScanTokens][KMAX], ks[2][MODE == 2 ? 1 : kScanTokens][KMAX], ds[2][MODE == 3 ? 1 : kScanTokens][KMAX];
     __shared__ __align__(16) float as[2][MODE == 1 ? kScanTokens : 1][KMAX], vs[2][kScanTokens][kCols], us[KMAX];
     __shared__ float is[2][kScanTokens];                                // MODE 1: 1 / (|k|^2 + 1e-6) of the staged tokens
@@ -194,6 +199,19 @@ state_scan_kernel(ScanInput r, ScanInput k, ScanInput v, ScanInput d, ScanInput 
                         else acc0 = fmaf(rv[e], S[ii], acc0);
                     }
                 }
+            } else if (MODE == 4) {
+#pragma unroll
+                for (int c4 = 0; c4 < RPT / 4; ++c4) {
+                    const float4 rr = r4[c4 * kSplit], kk = k4[c4 * kSplit], dd = d4[c4 * kSplit];
+                    const float rv[4] = {rr.x, rr.y, rr.z, rr.w}, kv4[4] = {kk.x, kk.y, kk.z, kk.w}, dv[4] = {dd.x, dd.y, dd.z, dd.w};
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const int ii = c4 * 4 + e;
+                        S[ii] = fmaf(dv[e], S[ii], kv4[e] * vj);
+                        if (e & 1) acc1 = fmaf(rv[e], S[ii], acc1);
+                        else acc0 = fmaf(rv[e], S[ii], acc0);
+                    }
+                }
             } else if (MODE == 2) {
 #pragma unroll
                 for (int c4 = 0; c4 < RPT / 4; ++c4) {
@@ -240,7 +258,7 @@ state_scan_kernel(ScanInput r, ScanInput k, ScanInput v, ScanInput d, ScanInput 
             float acc = acc0 + acc1;
 #pragma unroll
             for (int o = 1; o < kSplit; o <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-            if (live && q == 0) out[(size_t)(tb + tt) * N * KV + col] = acc;
+            if (live && q == 0) out[(size_t)(tb + tt) * N * KV + col] = MODE == 4 ? acc * out_scale : acc;
         }
         __syncthreads();                                                  // before the next copies overwrite this half
     }
@@ -341,15 +359,47 @@ retention_prepare_kernel(float* __restrict__ q, int ld_q, float* __restrict__ k,
     for (int c = rot_dims + lane; c < K; c += 32) kh[c] *= k_scale;
 }
 
+constexpr int kDecayThreads = 128, kDecayTokens = 8;
+
+// Decays from a low-rank projection: a[t][c] = sigmoid(u_t . w2[c] + b[c])^(1/tau) = exp(log sigmoid(.) / tau), for M channels and
+// hidden vectors u of r numbers, everything in fp32.  w2t [r, M] (transposed: neighbouring threads read neighbouring channels).
+// One CTA per (8 tokens, 128 channels).
+__global__ void __launch_bounds__(kDecayThreads)
+lowrank_decay_kernel(ScanInput u, const float* __restrict__ w2t, const float* __restrict__ b, float* __restrict__ a, int T, int r, int M,
+                     float inv_tau) {
+    extern __shared__ float us[];                     // [kDecayTokens][r]
+    forge::pdl_wait();             // (no early word: the scan follows, see scan_gates_kernel)
+    const int t0 = blockIdx.x * kDecayTokens, nt = min(kDecayTokens, T - t0);
+    for (int i = threadIdx.x; i < kDecayTokens * r; i += kDecayThreads) {
+        const int tt = i / r;
+        us[i] = tt < nt ? u.p[(size_t)(t0 + tt) * u.ld + i % r] : 0.f;
+    }
+    __syncthreads();
+    const int c = blockIdx.y * kDecayThreads + threadIdx.x;
+    if (c >= M) return;
+    float acc[kDecayTokens];
+#pragma unroll
+    for (int tt = 0; tt < kDecayTokens; ++tt) acc[tt] = b[c];
+#pragma unroll 8
+    for (int k = 0; k < r; ++k) {
+        const float w = w2t[(size_t)k * M + c];
+#pragma unroll
+        for (int tt = 0; tt < kDecayTokens; ++tt) acc[tt] = fmaf(us[tt * r + k], w, acc[tt]);
+    }
+#pragma unroll
+    for (int tt = 0; tt < kDecayTokens; ++tt)
+        if (tt < nt) a[(size_t)(t0 + tt) * M + c] = expf((fminf(acc[tt], 0.f) - log1pf(expf(-fabsf(acc[tt])))) * inv_tau);
+}
+
 template <int MODE, typename TA>
 cudaError_t launch_scan(int kmax, dim3 grid, cudaStream_t stream, ScanInput r, ScanInput k, ScanInput v, ScanInput d, ScanInput a,
                         const float* bonus, const float* inv, float* state, long long stride, const int32_t* q_start, const int32_t* slots,
-                        float* out, const TA* last_in, int W, long long prev_off, int N, int K, int KV, int vec) {
+                        float* out, const TA* last_in, int W, long long prev_off, int N, int K, int KV, int vec, float out_scale = 1.0f) {
 #define FORGE_SCAN_CASE(KM)                                                                                                  \
     case KM:                                                                                                                 \
         return forge::launch(state_scan_kernel<KM, MODE, TA>, grid, dim3(kScanThreads), 0, stream, 1, r, k, v, d, a, bonus, inv, state, \
-                             stride, q_start, slots, out, last_in, W, prev_off, N, K, KV, vec);
-    if constexpr (MODE == 2 || MODE == 3) {   // the gated write stages no keys, retention no decays: heads of up to 256 key channels fit
+                             stride, q_start, slots, out, last_in, W, prev_off, N, K, KV, vec, out_scale);
+    if constexpr (MODE >= 2) {   // the gated write stages no keys, retention no decays: heads of up to 256 key channels fit
         switch (kmax) {
             FORGE_SCAN_CASE(192) FORGE_SCAN_CASE(256)
             default: break;
@@ -443,6 +493,32 @@ extern "C" int forge_retention_scan(float* q, int ld_q, float* k, int ld_k, cons
     e = launch_scan<3, float>(kmax, grid, stream, Q, Kk, V, D, D, nullptr, nullptr, state, state_stride, q_start, slots, out, nullptr, 0, 0,
                               N, K, KV, vec);
     return forge::check_launch("retention_scan", e);
+}
+
+// Gated linear attention over the step's tokens: decays a = sigmoid(u . w2 + b)^(1/tau) per key channel into `decay` (fp32 [T, N*K]
+// scratch), then S <- diag(a) S + k v^T, out = q_scale S^T q per head.  q, k, v fp32 (row t at p + t * ld, head n's channels at
+// columns n*K .. or n*KV ..); u fp32 rows of ld_u with r hidden numbers; w2t fp32 [r, N*K], b fp32 [N*K]; out fp32 [T, N*KV]; a
+// head's state is [K, KV].
+extern "C" int forge_gla_scan(const float* q, int ld_q, const float* k, int ld_k, const float* v, int ld_v, const float* u, int ld_u, int r,
+                              const float* w2t, const float* b, float inv_tau, float q_scale, float* decay, float* state,
+                              long long state_stride, const int32_t* q_start, const int32_t* slots, float* out, int T, int S, int N, int K,
+                              int KV, cudaStream_t stream) {
+    if (T < 0 || S < 0 || N <= 0 || K <= 0 || KV <= 0 || r <= 0 || ld_u < r) return forge::fail(FORGE_ERR_ARG, "gla_scan: bad sizes S=%d N=%d K=%d V=%d r=%d", S, N, K, KV, r);
+    if (K > 256) return forge::fail(FORGE_ERR_UNSUPPORTED, "gla_scan: heads of %d key channels (at most 256)", K);
+    if (sizeof(float) * kDecayTokens * (size_t)r > 48 * 1024) return forge::fail(FORGE_ERR_UNSUPPORTED, "gla_scan: a hidden layer of %d numbers", r);
+    if (state_stride < (long long)N * K * KV) return forge::fail(FORGE_ERR_ARG, "gla_scan: state rows are too short");
+    if (S == 0 || T == 0) return FORGE_OK;
+    cudaError_t e = forge::launch(lowrank_decay_kernel, dim3((T + kDecayTokens - 1) / kDecayTokens, (N * K + kDecayThreads - 1) / kDecayThreads),
+                                  dim3(kDecayThreads), sizeof(float) * kDecayTokens * r, stream, 1, ScanInput{u, ld_u}, w2t, b, decay, T, r, N * K, inv_tau);
+    if (e != cudaSuccess) return forge::check_launch("gla_scan (decays)", e);
+    const int kmax = K <= 128 ? (K + 31) / 32 * 32 : (K <= 192 ? 192 : 256);
+    const dim3 grid(S, N, (KV + kCols - 1) / kCols);
+    ScanInput Q{q, ld_q}, Kk{k, ld_k}, V{v, ld_v}, D{decay, N * K};
+    auto aligned = [](const float* p, int ld) { return ((uintptr_t)p & 15) == 0 && ld % 4 == 0; };
+    const int vec = (K % 4 == 0 && aligned(q, ld_q) && aligned(k, ld_k) && aligned(decay, N * K)) ? 1 : 0;
+    e = launch_scan<4, float>(kmax, grid, stream, Q, Kk, V, D, D, nullptr, nullptr, state, state_stride, q_start, slots, out, nullptr, 0, 0, N,
+                              K, KV, vec, q_scale);
+    return forge::check_launch("gla_scan", e);
 }
 
 // h, out of type dtype: [T, W] and [n_mix, T, W]; mu fp32 [n_mix, W]; the kept row of request s: state + slots[s] * stride + prev_off.

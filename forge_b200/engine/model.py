@@ -40,6 +40,9 @@ class Model:
             if plan.streams < 1 or plan.add_embedding_before or type(self.final_norm) is not RMSNorm:
                 raise ConfigError("a stream kept as several copies needs an RMS norm at the end and no embedding added on the way")
             self._ones = None
+        if plan.depth_average and (plan.streams != 1 or plan.add_embedding_before or getattr(self.embedding, "needs_batch", False)
+                                   or plan.schedule != list(range(n))):
+            raise ConfigError("a stream averaged over the depth is one stream from an embedding without state through layers that run once, in order")
         self.loaded = False
         self._fused = None
         self._replay_ok, self._replay_from, self._replay_tensors = False, 0, []
@@ -131,7 +134,7 @@ class Model:
         self._fused = None
         sched = self.plan.schedule
         if self.rt.full_precision or not sched or sched != list(range(len(self.blocks))) or self.plan.add_embedding_before \
-                or self.plan.streams != 1:
+                or self.plan.streams != 1 or self.plan.depth_average:
             return False
         descs = [b.fused_decode() if hasattr(b, "fused_decode") else None for b in self.blocks]
         if any(d is None for d in descs):
@@ -181,7 +184,13 @@ class Model:
         ``embedding_cache`` what the embedding keeps (``embedding_cache_spec``).
         Returns fp32 logits [R,V] at ``batch.logits_rows`` (None if no row is wanted).  ``workspace``: the open
         StepWorkspace that the kernels' outputs are cut from; a layer's share of it is given back after the layer."""
-        if getattr(self.embedding, "needs_batch", False):
+        depth = self.plan.depth_average
+        if depth:
+            # planes of the stream's history: the embedding output first, the stream itself last
+            residual = kernels.new_tensor((len(self.plan.schedule) + 1, batch.num_tokens, self.plan.hidden_size), torch.float32,
+                                          batch.token_ids.device)
+            self.embedding.forward(batch.token_ids, status=batch.status, out=residual[0])
+        elif getattr(self.embedding, "needs_batch", False):
             residual = self.embedding.forward_step(batch, embedding_cache)
         else:
             residual = self.embedding.forward(batch.token_ids, status=batch.status)
@@ -205,9 +214,12 @@ class Model:
                 if replay is not None:
                     replay.run(self._replay_tensors[pos] + [position_caches[pos].kv])
                     continue
-                if S != 1:
+                if S != 1 or depth:
                     # a block may leave the next block's first input in the same pass as its own last write to the copies
                     batch.shared["following_block"] = self.blocks[self.plan.schedule[pos + 1]] if pos + 1 < len(self.plan.schedule) else None
+                if depth:
+                    # ... and the last one the head's input: the model's norm of the wanted rows
+                    batch.shared["last_norm"] = (self.final_norm, batch.logits_rows) if pos + 1 == len(self.plan.schedule) else None
                 # one layer's launches are noted and repeated for the layers after it (what the whole step shares,
                 # tile lists and the table of angles, is made inside the first layer: those launches are marked
                 # and stay out of the notes)
@@ -229,6 +241,10 @@ class Model:
             # the last norm reads the sum of the copies
             x = kernels.streams_mix(residual, S, in_next=self._ones, w_next=self.final_norm.weight, eps=self.final_norm.eps,
                                     out_dtype=self.rt.dtype, rows=batch.logits_rows)
+        elif depth:
+            x = batch.shared.pop("last_input", None)
+            if x is None:
+                x = self.final_norm.forward(residual[-1], rows=batch.logits_rows)
         else:
             x = self.final_norm.forward(residual, rows=batch.logits_rows)
         if workspace is None:

@@ -38,7 +38,8 @@ _SIGNATURES = {
         "forge_streams_expand": [_P, _P, _I, _I, _I, _P],
         "forge_streams_mix": [_P] * 7 + [_I, _P, _I, _I, _I, _F, _P],
         "forge_layernorm": [_P, _P, _P, _P, _I, _P, _I, _I, _F, _P],
-        "forge_act_rows": [_P, _I, _P, _I, _I, _I, _I, _P],
+        "forge_act_rows": [_P, _I, _P, _I, _I, _I, _I, _F, _F, _P],
+        "forge_depth_step": [_P, _LL, _I, _I, _I, _I] + [_P] * 4 + [_I, _I, _I, _P, _P, _I, _F, _P, _I, _P, _I, _I, _P],
         "forge_rmsnorm": [_P, _P, _P, _I, _P, _I, _I, _F, _P],
         "forge_rmsnorm_pair": [_P, _P, _P, _P, _P, _I, _I, _I, _F, _P],
         "forge_rope_kv_write": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _P, _P],
@@ -53,7 +54,7 @@ _SIGNATURES = {
         "forge_history_add": [_P, _P, _P, _P, _I, _I, _P],
     },
     "gemm_sm100": {
-        "forge_gemm_sm100": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _P],
+        "forge_gemm_sm100": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _F, _F, _P],
         "forge_gemm_sm100_set_workspace": [_P, ctypes.c_longlong],
         "forge_gemm_sm100_qkv_rope": [_P] * 8 + [_I] * 7 + [_P],
     },
@@ -78,11 +79,12 @@ _SIGNATURES = {
         "forge_token_shift": [_P, _P, _LL, _LL, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P],
         "forge_head_finish": [_P, _P, _P, _I, _P, _I, _I, _I, _I, _F, _I, _F, _I, _LL, _P],
         "forge_tanh_rows": [_P, _I, _P, _I, _I, _I, _P],
+        "forge_gla_scan": [_P, _I] * 4 + [_I, _P, _P, _F, _F, _P, _P, _LL, _P, _P, _P, _I, _I, _I, _I, _I, _P],
         "forge_retention_scan": [_P, _I, _P, _I, _P, _I, _P, _P, _I, _F, _P, _P, _LL, _P, _P, _P, _I, _I, _I, _I, _I, _P],
     },
     "latent": {
-        "forge_latent_prepare": [_P, _I, _P, _P, _P, _F, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _P],
-        "forge_head_linear": [_P, _I, _LL, _I, _P, _P, _I, _LL, _I, _P, _P, _F, _I, _I, _I, _I, _I, _I, _P, _LL, _P],
+        "forge_latent_prepare": [_P, _I, _P, _P, _P, _F, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P],
+        "forge_head_linear": [_P, _I, _LL, _I, _P, _P, _I, _LL, _I, _P, _P, _F, _I, _I, _I, _I, _I, _I, _P, _LL, _I, _I, _I, _P],
         "forge_latent_attention": [_P] * 8 + [_I] * 8 + [_F, _I, _I, _I, _P, _P],
         "forge_latent_mma_supports": [_I] * 4,
         "forge_latent_mma_heads": [_I],
@@ -634,29 +636,72 @@ def rmsnorm(x, weight, eps, out_dtype, rows=None, out=None):
 
 
 def layernorm(x, weight, bias, eps, out_dtype, rows=None):
-    """y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b over the last dim of float32 x [T,H]; ``rows`` (int32) picks rows."""
+    """y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b over the last dim of float32 x [T,H] (``bias`` None: no b); ``rows``
+    (int32) picks rows."""
     lib = library("core")
     H = x.shape[-1]
     R = x.shape[0] if rows is None else rows.numel()
-    if weight.numel() != H or bias.numel() != H:
-        raise KernelError(f"layernorm: weight and bias have {weight.numel()} and {bias.numel()} elements, rows have {H}")
+    if weight.numel() != H or (bias is not None and bias.numel() != H):
+        raise KernelError(f"layernorm: weight and bias have {weight.numel()} and {None if bias is None else bias.numel()} elements, rows have {H}")
     out = new_tensor((R, H), out_dtype, x.device)
     _check(lib, lib.forge_layernorm(_need(x, "x", torch.float32, 2), _need(weight, "weight", torch.float32),
-                                    _need(bias, "bias", torch.float32), _need(out, "out", out_dtype), dtype_code(out_dtype),
+                                    _opt(bias, "bias", torch.float32), _need(out, "out", out_dtype), dtype_code(out_dtype),
                                     _opt(rows, "rows", torch.int32), R, H, float(eps), _stream()), "layernorm")
     return out
 
 
-ACTIVATIONS = {"gelu": 0, "gelu_tanh": 1, "silu": 2}
+ACTIVATIONS = {"gelu": 0, "gelu_tanh": 1, "silu": 2, "xielu": 3}
 
 
-def act_rows(x, out_dtype, activation):
-    """activation(x) of float32 x [T,n] in ``out_dtype``: "gelu" (the exact one, with erf), "gelu_tanh", "silu"."""
+def act_rows(x, out_dtype, activation, numbers=None):
+    """activation(x) of float32 x [T,n] in ``out_dtype``: "gelu" (the exact one, with erf), "gelu_tanh", "silu", or "xielu" with
+    ``numbers`` = (a, b): a x^2 + x/2 above zero, b (exp(x) - 1 - x) + x/2 below."""
+    a, b = _act_numbers(activation, numbers)
     lib = library("core")
     T, n = x.shape
     out = new_tensor((T, n), out_dtype, x.device)
     _check(lib, lib.forge_act_rows(_need(x, "x", torch.float32, 2), n, _need(out, "out", out_dtype), dtype_code(out_dtype), T, n,
-                                   ACTIVATIONS[activation], _stream()), "act_rows")
+                                   ACTIVATIONS[activation], a, b, _stream()), "act_rows")
+    return out
+
+
+def _act_numbers(activation, numbers):
+    if (activation == "xielu") != (numbers is not None):
+        raise KernelError("the activation xielu takes two numbers, the others none")
+    return (0.0, 0.0) if numbers is None else (float(numbers[0]), float(numbers[1]))
+
+
+def depth_step(planes, n, x_plane, y1, y2=None, gates=None, weights=None, new_plane=-1, s_plane=-1, next_norm=None, out_dtype=None, rows=None,
+               out=None):
+    """What a layer does to a stream that is averaged over the depth.  ``planes`` fp32 [P, T, W]: plane j is what layer j - 1 left
+    (0: the embedding output).  With x = planes[x_plane] and the gates sigmoid(z1), sigmoid(z2)
+        X_new = x + (y1 * sigmoid(z1) + y2 * sigmoid(z2)),   s = sum_j weights[j] planes[j] + weights[n-1] X_new  (j < n - 1)
+    X_new goes to planes[new_plane] and s to planes[s_plane] (-1: nowhere).  ``gates`` = (fp32 matrix, first column of z1, first
+    column of z2), None: no gates; ``y2`` None: one sublayer; ``weights`` None (n = 0): s = X_new.  ``next_norm`` = ("layer" | "rms",
+    weight, bias or None, eps): returns that norm of s in ``out_dtype`` ([T, W], or [R, W] with ``rows`` int32 [R], which then
+    restricts everything to those tokens), written into ``out`` if given; None without it."""
+    lib = library("core")
+    P, T, W = planes.shape
+    R = T if rows is None else rows.numel()
+    if tuple(y1.shape) != (T, W) or (y2 is not None and tuple(y2.shape) != (T, W)) or max(x_plane, new_plane, s_plane, n - 2) >= P \
+            or (0 if weights is None else weights.numel()) != n or (gates is not None and gates[0].shape[0] != T):
+        raise KernelError(f"depth_step: planes {tuple(planes.shape)}, outputs {tuple(y1.shape)}, {n} weights do not fit")
+    zp, z1, z2 = (None, 0, 0) if gates is None else gates
+    kind, w, b, eps = next_norm if next_norm is not None else ("layer", None, None, 0.0)
+    if w is None:
+        out = None
+    else:
+        if w.numel() != W or (b is not None and b.numel() != W):
+            raise KernelError(f"depth_step: the norm's weights do not fit rows of {W}")
+        out = new_tensor((R, W), out_dtype, planes.device) if out is None else out
+        if tuple(out.shape) != (R, W):
+            raise KernelError(f"depth_step: the output given is {tuple(out.shape)}, the normed rows are {(R, W)}")
+    _check(lib, lib.forge_depth_step(
+        _need(planes, "planes", torch.float32, 3), T * W, n, x_plane, new_plane, s_plane, _opt(weights, "weights", torch.float32),
+        _need(y1, "y1", torch.float32, 2), _opt(y2, "y2", torch.float32), _opt(zp, "gates", torch.float32), 0 if zp is None else zp.shape[1],
+        int(z1), int(z2), _opt(w, "w", torch.float32), _opt(b, "b", torch.float32), {"rms": 0, "layer": 1}[kind], float(eps),
+        _opt(out, "out", out_dtype), dtype_code(out_dtype) if out is not None else F32, _opt(rows, "rows", torch.int32), R, W, _stream()),
+        "depth_step")
     return out
 
 
@@ -1084,46 +1129,82 @@ def retention_scan(q, k, v, batch, freq, k_scale, decay, state, N, K, KV):
     return out
 
 
+def gla_scan(q, k, v, hidden, rank, w2t, bias, tau, batch, state, N, K, KV):
+    """Gated linear attention over the step's tokens, request by request, from and into ``state`` fp32 [slots, N*K*KV]: decays
+    a = sigmoid(hidden . w2 + bias)^(1/tau) per key channel (``w2t`` fp32 [rank, N*K]), S <- diag(a) S + k v^T, out = K^-1/2 S^T q per
+    head.  q, k, v, hidden: (fp32 matrix, first column) pairs; returns fp32 [T, N*KV]."""
+    lib = library("mixers")
+    T = q[0].shape[0]
+    if tuple(w2t.shape) != (rank, N * K) or bias.numel() != N * K or not tau > 0.0:
+        raise KernelError(f"gla_scan: w2 {tuple(w2t.shape)}, {bias.numel()} biases and tau {tau} do not fit {N} heads of {K}, rank {rank}")
+    decay = new_tensor((T, N * K), torch.float32, q[0].device)
+    out = new_tensor((T, N * KV), torch.float32, q[0].device)
+    (qp, ql), (kp, kl), (vp, vl), (up, ul) = _cols(*q), _cols(*k), _cols(*v), _cols(*hidden)
+    _check(lib, lib.forge_gla_scan(
+        qp, ql, kp, kl, vp, vl, up, ul, int(rank), _need(w2t, "w2t", torch.float32, 2), _need(bias, "bias", torch.float32), 1.0 / float(tau),
+        float(K) ** -0.5, _need(decay, "decay", torch.float32), _need(state, "state", torch.float32, 2), state.shape[1],
+        _need(batch.q_start, "q_start", torch.int32), _need(batch.slots, "slots", torch.int32), _need(out, "out", torch.float32), T,
+        batch.num_requests, N, K, KV, _stream()), "gla_scan")
+    count_launches(1)              # the kernel that makes the decays
+    return out
+
+
 # ---------------------------------------------------------------------------------------------- latent attention
 
 LATENT_KEYS_PER_CHUNK = 32          # fixed: a token's sums must not depend on the step's shape
 
 
-def latent_prepare(proj, batch, slot_mapping, cache, freq, amp, wq, wc, Cq, C, R, eps, act_dtype):
-    """proj fp32 [T, Cq (+ C + R)]: the query latent normed (weight ``wq``) -> [T, Cq] in ``act_dtype``; with C > 0 the normed
-    key/value latent (weight ``wc``) and the rotated shared key part go to ``slot_mapping`` in ``cache`` (rows of C + R)."""
+def latent_prepare(proj, batch, slot_mapping, cache, freq, amp, wq, wc, Cq, C, R, eps, act_dtype, halves=False):
+    """proj fp32 [T, Cq (+ C + R)], or (matrix, first column): the query latent normed (weight ``wq``) -> [T, Cq] in ``act_dtype``
+    (Cq = 0: none, returns None); with C > 0 the normed key/value latent (weight ``wc``) and the rotated shared key part go to
+    ``slot_mapping`` in ``cache`` (rows of C + R).  ``halves``: the rotation pairs channel i with i + R/2 instead of 2i with 2i + 1."""
     lib = library("latent")
+    proj, col = proj if isinstance(proj, tuple) else (proj, 0)
     T, ld = proj.shape
-    cq = new_tensor((T, Cq), act_dtype, proj.device)
     store = C > 0 and cache is not None and slot_mapping is not None
+    if Cq == 0 and not store:
+        return None
+    if ld < col + Cq + (C + R if store else 0):
+        raise KernelError(f"latent_prepare: rows of {ld} numbers from column {col} do not hold {Cq} + {C} + {R}")
+    cq = new_tensor((T, Cq), act_dtype, proj.device) if Cq else None
     if store and cache.dtype != act_dtype:
         raise KernelError("latent_prepare: cache and activation dtypes differ")
     _check(lib, lib.forge_latent_prepare(
-        _need(proj, "proj", torch.float32, 2), ld, _need(batch.positions, "positions", torch.int32),
+        _cols(proj, col)[0], ld, _need(batch.positions, "positions", torch.int32),
         _need(slot_mapping, "slot_mapping", torch.int32) if store else None, _opt(freq, "freq", torch.float32), float(amp),
-        _need(wq, "wq", torch.float32), _opt(wc, "wc", torch.float32), _need(cq, "cq", act_dtype), _need(cache, "cache") if store else None,
-        dtype_code(act_dtype), T, Cq, C if ld > Cq else 0, R, float(eps), _stream()), "latent_prepare")
+        _opt(wq, "wq", torch.float32), _opt(wc, "wc", torch.float32), _opt(cq, "cq", act_dtype), _need(cache, "cache") if store else None,
+        dtype_code(act_dtype), T, Cq, C if store else 0, R, float(eps), 1 if halves else 0, _stream()), "latent_prepare")
     return cq
 
 
-def head_linear(x, w, H, K, N, out_dtype, R=0, positions=None, freq=None, amp=1.0, simt=False, gate=None):
-    """out[t, h, :N] = sum_k x[t, h, k] w[h, k, :] for the H heads of x [T, H*(K+R)] (fp32 or the weights' type); with R > 0 a head's
-    last R channels are rotated by position * freq (channel 2i with 2i+1, cos and sin times ``amp``) and follow the N outputs.
-    w [H, K, N] in ``out_dtype``; returns [T, H*(N+R)] in ``out_dtype``.  bfloat16 weights go to the tensor cores (an fp32 x rounded to
-    bfloat16 on the way) unless ``simt`` asks for fp32 multiply-adds on the inputs as they are.  ``gate`` = (fp32 matrix, first
-    column): the outputs are multiplied by the sigmoid of the H*N numbers from that column of the token's row."""
+def head_linear(x, w, H, K, N, out_dtype, R=0, positions=None, freq=None, amp=1.0, simt=False, gate=None, halves=False, out=None):
+    """out[t, h, :N] = sum_k x[t, h, k] w[h, k, :] for the H heads of x [T, H*(K+R)] (fp32 or the weights' type; or (matrix, first
+    column), fp32); with R > 0 a head's last R channels are rotated by position * freq (channel 2i with 2i+1, with ``halves`` i with
+    i + R/2; cos and sin times ``amp``) and follow the N outputs.  w [H, K, N] in ``out_dtype``; returns [T, H*(N+R)] in ``out_dtype``
+    (or writes them into ``out`` = (matrix, first column)).  bfloat16 weights go to the tensor cores (an fp32 x rounded to bfloat16 on
+    the way) unless ``simt`` asks for fp32 multiply-adds on the inputs as they are.  ``gate`` = (fp32 matrix, first column) or (fp32
+    matrix, first column, "head"): the outputs are multiplied by the sigmoid of the H*N numbers from that column of the token's row,
+    or of the H numbers there, one per head."""
     lib = library("latent")
-    gate_ptr, gate_ld = (None, 0) if gate is None else _cols(gate[0], gate[1])
-    if gate is not None and (R or gate[0].shape[0] != x.shape[0] or gate[0].shape[1] < gate[1] + H * N):
-        raise KernelError("head_linear: a gate wants rows of the step's tokens with H*N columns, and no rotated channels")
-    T = x.shape[0]
-    if x.shape[1] != H * (K + R) or tuple(w.shape) != (H, K, N) or w.dtype != out_dtype:
+    gate_ptr, gate_ld, gate_hs, gate_cs = None, 0, 0, 0
+    if gate is not None:
+        gate_hs, gate_cs = (1, 0) if gate[2:] == ("head",) else (N, 1)
+        gate_ptr, gate_ld = _cols(gate[0], gate[1])
+    T = (x[0] if isinstance(x, tuple) else x).shape[0]
+    if gate is not None and (R or gate[0].shape[0] != T or gate[0].shape[1] < gate[1] + (H if gate_hs == 1 and gate_cs == 0 else H * N)):
+        raise KernelError("head_linear: a gate wants rows of the step's tokens with H*N columns (or H), and no rotated channels")
+    if isinstance(x, tuple):
+        (x, col), fits = x, x[0].shape[1] >= x[1] + H * (K + R)
+        x_ptr, x_ld = _cols(x, col)
+    else:
+        x_ptr, x_ld, fits = _need(x, "x", ndim=2), x.shape[1], x.shape[1] == H * (K + R)
+    if not fits or tuple(w.shape) != (H, K, N) or w.dtype != out_dtype:
         raise KernelError(f"head_linear: x {tuple(x.shape)}, w {tuple(w.shape)} {w.dtype} do not fit {H} heads of {K}+{R} -> {N}")
-    out = new_tensor((T, H * (N + R)), out_dtype, x.device)
+    out, out_ptr, out_ld = _out_slice(out, H * (N + R), T, out_dtype, x.device)
     _check(lib, lib.forge_head_linear(
-        _need(x, "x", ndim=2), dtype_code(x.dtype), H * (K + R), K + R, _need(w, "w"), _need(out, "out", out_dtype), dtype_code(out_dtype),
-        H * (N + R), N + R, _opt(positions, "positions", torch.int32), _opt(freq, "freq", torch.float32), float(amp), T, H, K, N, R,
-        1 if simt else 0, gate_ptr, gate_ld, _stream()), "head_linear")
+        x_ptr, dtype_code(x.dtype), x_ld, K + R, _need(w, "w"), out_ptr, dtype_code(out_dtype),
+        out_ld, N + R, _opt(positions, "positions", torch.int32), _opt(freq, "freq", torch.float32), float(amp), T, H, K, N, R,
+        1 if simt else 0, gate_ptr, gate_ld, gate_hs, gate_cs, 1 if halves else 0, _stream()), "head_linear")
     return out
 
 
@@ -1699,18 +1780,19 @@ def paged_attention(q, kv_cache, group_batch, batch, n_heads, n_kv_heads, head_d
 
 EPILOGUES = {"none": 0, "accumulate": 1, "cast": 2, "swiglu": 3, "geglu": 5}
 GELU_GATE_VARIANT = {"FORGE_GATE_GELU": 1}
-GELU_CAST_VARIANT = {"FORGE_CAST_ACT": 1}        # the library whose bfloat16 store applies the exact gelu first
+# libraries whose bfloat16 store applies an activation first: the exact gelu, xIELU with the call's two numbers
+CAST_VARIANTS = {"gelu": {"FORGE_CAST_ACT": 1}, "xielu": {"FORGE_CAST_ACT": 2}}
 
 
-def gemm_sm100(x, w, bias=None, accumulate_into=None, epilogue="none", tile_n=0, status=None, out=None, live=None):
+def gemm_sm100(x, w, bias=None, accumulate_into=None, epilogue="none", tile_n=0, status=None, out=None, live=None, numbers=None):
     """bf16 x [M,K] . w [N,K]^T on the tcgen05 tensor cores, fp32 accumulation.
     epilogue "none": fp32 [M,N] (added into ``accumulate_into`` when given); "cast": bf16 [M,N];
     "swiglu": bf16 [M,N/2] = silu(y[:,2j]) * y[:,2j+1]; "geglu": the same with the tanh form of gelu; "gelu": bf16 [M,N] =
-    y/2 (1 + erf(y / sqrt 2)).
+    y/2 (1 + erf(y / sqrt 2)); "xielu": bf16 [M,N], see ``act_rows`` (``numbers`` its two numbers).
     ``live``: an int32 device word (a one-element tensor) written by an earlier kernel; where it holds 0 the product is skipped on the
     device, nothing read and nothing written."""
     # the gelu gate lives in a variant of the library of its own, so that the silu epilogues stay as short as they were
-    lib = library("gemm_sm100", GELU_GATE_VARIANT if epilogue == "geglu" else GELU_CAST_VARIANT if epilogue == "gelu" else None)
+    lib = library("gemm_sm100", GELU_GATE_VARIANT if epilogue == "geglu" else CAST_VARIANTS.get(epilogue))
     (M, K), (N, K2) = x.shape, w.shape
     if K != K2:
         raise KernelError(f"gemm_sm100: x {tuple(x.shape)} does not match w {tuple(w.shape)}")
@@ -1721,7 +1803,7 @@ def gemm_sm100(x, w, bias=None, accumulate_into=None, epilogue="none", tile_n=0,
             out = new_tensor((M, N), torch.float32, x.device) if out is None else out
             code = EPILOGUES["none"]
         want_shape, want_dtype = (M, N), torch.float32
-    elif epilogue in ("cast", "gelu"):
+    elif epilogue in ("cast", "gelu", "xielu"):
         out = new_tensor((M, N), torch.bfloat16, x.device) if out is None else out
         code, want_shape, want_dtype = EPILOGUES["cast"], (M, N), torch.bfloat16
     elif epilogue in ("swiglu", "geglu"):
@@ -1736,7 +1818,8 @@ def gemm_sm100(x, w, bias=None, accumulate_into=None, epilogue="none", tile_n=0,
     _gemm_workspace(lib, x.device)
     _check(lib, lib.forge_gemm_sm100(_need(x, "x", torch.bfloat16, 2), _need(w, "w", torch.bfloat16, 2),
                                      _opt(bias, "bias", torch.float32), _need(out, "out", want_dtype),
-                                     _need(status, "status", torch.int32), M, N, K, code, int(tile_n), _opt(live, "live", torch.int32), _stream()),
+                                     _need(status, "status", torch.int32), M, N, K, code, int(tile_n), _opt(live, "live", torch.int32),
+                                     *_act_numbers(epilogue, numbers), _stream()),
            "gemm_sm100")
     return out
 

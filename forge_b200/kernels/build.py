@@ -20,9 +20,9 @@ CSRC = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))),
 
 LIBRARIES = {
     # embedding, norm, rotary + cache write, activation, fp32 GEMM, fp32/any-shape attention, sampling
-    # ... and a residual stream kept as several copies
+    # ... and a residual stream kept as several copies, or averaged over the depth
     "core": ["embedding.cu", "norm.cu", "rope_cache.cu", "activation.cu", "gemm_simt.cu",
-             "attention_simt.cu", "sampling.cu", "streams.cu"],
+             "attention_simt.cu", "sampling.cu", "streams.cu", "depth.cu"],
     # bf16 tcgen05 + TMA GEMM with fused epilogues
     "gemm_sm100": ["gemm_sm100.cu"],
     # bf16 tensor-core paged attention (mma.sync) for any head size, prompt portions and decode
@@ -156,4 +156,5 @@ def build_all(force=False):
             out[name] = build_library(name, force=force)
     out["gemm_sm100_gate_gelu1"] = build_library("gemm_sm100", force=force, defines={"FORGE_GATE_GELU": 1})
     out["gemm_sm100_cast_act1"] = build_library("gemm_sm100", force=force, defines={"FORGE_CAST_ACT": 1})
+    out["gemm_sm100_cast_act2"] = build_library("gemm_sm100", force=force, defines={"FORGE_CAST_ACT": 2})
     return out

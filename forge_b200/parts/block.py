@@ -12,6 +12,10 @@ model's last norm reads).  Around sublayer q (1: mixer, 2: feed-forward), with w
     u = sum_s in_q[s] x_s;   y = sublayer(norm_q(u));   x_t <- sum_s mix_q[s, t] x_s + out_q[t] y   (all t at once, from the old copies)
 in place of the residual sum.  A sublayer's write and the next sublayer's read and norm are one kernel, also across layers: where the
 model says which block runs next (``batch.shared["following_block"]``), a layer's last write leaves that block's first input.
+"parallel_depth":  with h = norm(x) for both sublayers,  X_new = x + g1 * mixer(h) + g2 * feed_forward(h),  g_q = sigmoid(Wg_q h + b_q) per
+channel, and what goes on is a weighted sum over the depth, x <- sum_j c[j] X_j of everything the layers have left so far (X_0: the
+embedding output).  The two gates ride in the mixer's input product; the gated sum, the average and the next layer's norm (after
+the last layer the model's norm, on the wanted rows) are one kernel.
 """
 from ..weights.loader import TensorSpec  # noqa: F401  (re-exported for part authors)
 from .base import Part, build_part, register_part
@@ -251,13 +255,9 @@ class HyperConnectionBlock(Part):
         if not isinstance(nxt, HyperConnectionBlock) or nxt.streams != S or nxt.rt.dtype != self.rt.dtype:
             kernels.streams_mix(residual, S, y=y, mix=w[f"{q}.mix"], out_w=w[f"{q}.out"])
             return
-        bufs = batch.shared.setdefault("stream_input_buffers", [None, None])
-        turn = batch.shared["stream_input_turn"] = 1 - batch.shared.get("stream_input_turn", 1)
-        if bufs[turn] is None:
-            bufs[turn] = kernels.new_tensor((y.shape[0], y.shape[1]), self.rt.dtype, y.device, whole_step=True)
         n1 = nxt.norms["mixer_in"]
         x = kernels.streams_mix(residual, S, y=y, mix=w[f"{q}.mix"], out_w=w[f"{q}.out"], in_next=nxt.weights["1.in"], w_next=n1.weight,
-                                eps=n1.eps, out_dtype=self.rt.dtype, out=bufs[turn])
+                                eps=n1.eps, out_dtype=self.rt.dtype, out=step_buffer(batch, y.shape[0], y.shape[1], self.rt.dtype, y.device))
         batch.shared["stream_input"] = (nxt, x)
 
     def forward(self, residual, batch, cache):
@@ -278,6 +278,103 @@ class HyperConnectionBlock(Part):
         self._last_write(residual, batch, y, 2)
 
 
+class ParallelDepthBlock(Part):
+    """``norms``: {"input": spec}.  ``residual`` is fp32 [runs + 1, T, W]: plane j is X_j, the last plane the stream x (which the first
+    run reads from X_0, and the last run's X is not kept).  How many planes there are before a layer's run is in the length of its
+    weights ``dwa`` [n]: it reads planes 0 .. n-2 and writes plane n-1.  ``layer_spec.block_params``: {"depth": n}.  The mixer must offer its
+    input product (``proj``, ``mix``, ``o``), the feed-forward return its output; tensors ``rg1``, ``rg1.b``, and ``rg2``, ``rg2.b`` with a
+    feed-forward."""
+    graph_safe = True
+    ROW_MULTIPLE = 8         # the shared product's rows are filled up to a multiple of this: aligned rows of its result
+
+    def sub_parts(self):
+        return [self.mixer, self.feed_forward, self.norm]
+
+    def __init__(self, rt, layer_spec):
+        from ..config.base import ConfigError
+        from .feedforward import NoFeedForward
+        self.rt = rt
+        self.mixer = build_part("mixer", layer_spec.mixer, rt)
+        self.feed_forward = build_part("feed_forward", layer_spec.feed_forward, rt)
+        self.norm = build_part("norm", layer_spec.norms["input"], rt)
+        self.depth = int((layer_spec.block_params or {}).get("depth", 0))
+        if self.depth < 2 or not hasattr(self.mixer, "mix") or not hasattr(self.norm, "fused"):
+            raise ConfigError("a layer whose stream is averaged over the depth needs weights of two planes at least, a mixer that "
+                              "offers its input product, and a layer norm or an RMS norm")
+        self.has_ff = type(self.feed_forward) is not NoFeedForward
+        self.proj = self.weights = None
+
+    def _children(self):
+        return [self.mixer, self.feed_forward, self.norm]
+
+    def tensor_specs(self):
+        W = self.norm.size
+        specs = {}
+        for part in self._children():
+            specs.update(part.tensor_specs())
+        for q in (1, 2):
+            # a layer without a feed-forward has no second gate; a file that carries its weights all the same is not refused
+            need = q == 1 or self.has_ff
+            specs.update({f"rg{q}": TensorSpec((W, W), required=need), f"rg{q}.b": TensorSpec((W,), required=need, role="bias")})
+        specs["dwa"] = TensorSpec((self.depth,), role="depth_mix")
+        return specs
+
+    def bind(self, tensors):
+        import torch
+        from .linear import Linear
+        for part in self._children():
+            part.bind({name: tensors[name] for name in part.tensor_specs() if name in tensors})
+        self.weights = self._vector_f32(tensors["dwa"])
+        # the gates and the mixer's inputs read the same h: one product, [gate 1 | gate 2 | the mixer's] (and rows of zeros at the end)
+        W, own = self.norm.size, self.mixer.proj
+        gates = [f"rg{q}" for q in ((1, 2) if self.has_ff else (1,))]
+        self.gate_cols = (0, W)
+        self.mixer_col = W * len(gates)
+        pad = -(self.mixer_col + own.out_features) % self.ROW_MULTIPLE
+        mats = [self._matrix(tensors[g]) for g in gates] + [own.weight, own.weight.new_zeros(pad, own.in_features)]
+        biases = [self._vector_f32(tensors[g + ".b"]) for g in gates]
+        own_bias = own.bias if own.bias is not None else torch.zeros(own.out_features, dtype=torch.float32, device=own.weight.device)
+        self.proj = Linear(torch.cat(mats, dim=0).contiguous(), torch.cat(biases + [own_bias, own_bias.new_zeros(pad)]), self.rt)
+        self.mixer.proj = None                         # the mixer's own copy is not needed any more
+
+    def forward(self, residual, batch, cache):
+        from .. import kernels
+        n, runs, T, W = self.depth, residual.shape[0] - 1, residual.shape[1], residual.shape[2]
+        x_plane = 0 if n == 2 else runs
+        left = batch.shared.pop("stream_input", None)          # (the block it is meant for, its input) from the layer before
+        h = left[1] if left is not None and left[0] is self else self.norm.forward(residual[x_plane])
+        p = self.proj.forward(h)
+        m = self.mixer.mix(p, self.mixer_col, batch, cache)
+        last = batch.shared.get("last_norm")                   # (the model's norm, the wanted rows) in the schedule's last run
+        if last is not None and last[1] is None:
+            return                                             # nothing reads what the last layer leaves: its cache is written
+        y1 = self.mixer.o.forward(m)
+        y2 = self.feed_forward.forward(h, None) if self.has_ff else None
+        following = batch.shared.get("following_block")
+        step = dict(gates=(p, *self.gate_cols), weights=self.weights, out_dtype=self.rt.dtype)
+        if last is not None and hasattr(last[0], "fused"):
+            x = kernels.depth_step(residual, n, x_plane, y1, y2, next_norm=last[0].fused(), rows=last[1], **step)
+            batch.shared["last_input"] = x
+            return
+        step.update(new_plane=n - 1 if n - 1 < runs else -1, s_plane=runs)
+        if isinstance(following, ParallelDepthBlock) and following.rt.dtype == self.rt.dtype:
+            x = kernels.depth_step(residual, n, x_plane, y1, y2, next_norm=following.norm.fused(), out=step_buffer(batch, T, W, self.rt.dtype, p.device),
+                                   **step)
+            batch.shared["stream_input"] = (following, x)
+        else:
+            kernels.depth_step(residual, n, x_plane, y1, y2, **step)
+
+
+def step_buffer(batch, T, W, dtype, device):
+    """One of two [T, W] buffers that live as long as the step, taken in turn: what a layer leaves for the next one."""
+    from .. import kernels
+    bufs = batch.shared.setdefault("stream_input_buffers", [None, None])
+    turn = batch.shared["stream_input_turn"] = 1 - batch.shared.get("stream_input_turn", 1)
+    if bufs[turn] is None:
+        bufs[turn] = kernels.new_tensor((T, W), dtype, device, whole_step=True)
+    return bufs[turn]
+
+
 def build_block(layer_spec, rt):
     from .base import _REGISTRY
     from ..config.base import ConfigError
@@ -292,3 +389,4 @@ register_part("block", "pre_norm", PreNormBlock, replace=True)
 register_part("block", "parallel", ParallelBlock, replace=True)
 register_part("block", "sandwich", SandwichBlock, replace=True)
 register_part("block", "hyper_connections", HyperConnectionBlock, replace=True)
+register_part("block", "parallel_depth", ParallelDepthBlock, replace=True)

@@ -52,8 +52,9 @@ class GeGLU(SwiGLU):
 
 
 class DenseFeedForward(Part):
-    """Ungated feed-forward:  residual += act(x.Wu^T) . Wd^T; ``activation``: "gelu" (the exact one, with erf),
-    "gelu_tanh" or "silu"; ``names``: the two matrices' tensor names."""
+    """Ungated feed-forward:  residual += act(x.Wu^T) . Wd^T; ``activation``: "gelu" (the exact one, with erf), "gelu_tanh", "silu", or
+    "xielu", whose two numbers (p, q) are a tensor of their own (``names["act"]``): the curvatures are softplus(p) above zero and
+    1/2 + softplus(q) below; ``names``: the tensors' names."""
     graph_safe = True
 
     def __init__(self, rt, hidden_size, intermediate_size, activation="gelu", names=None):
@@ -62,20 +63,27 @@ class DenseFeedForward(Part):
             from ..config.base import ConfigError
             raise ConfigError(f"feed-forward activation must be one of {sorted(kernels.ACTIVATIONS)}, got {activation!r}")
         self.rt, self.hidden_size, self.intermediate_size, self.activation = rt, hidden_size, intermediate_size, activation
-        self.names = {"up": "mlp.up", "down": "mlp.down", **(names or {})}
-        self.up = self.down = None
+        self.names = {"up": "mlp.up", "down": "mlp.down", "act": "mlp.act", **(names or {})}
+        self.up = self.down = self.numbers = None
 
     def tensor_specs(self):
         n, H, I = self.names, self.hidden_size, self.intermediate_size
-        return {n["up"]: TensorSpec((I, H)), n["down"]: TensorSpec((H, I))}
+        specs = {n["up"]: TensorSpec((I, H)), n["down"]: TensorSpec((H, I))}
+        if self.activation == "xielu":
+            specs[n["act"]] = TensorSpec((2,), role="bias")
+        return specs
 
     def bind(self, tensors):
         self.up = Linear(self._matrix(tensors[self.names["up"]]), None, self.rt)
         self.down = Linear(self._matrix(tensors[self.names["down"]]), None, self.rt)
+        if self.activation == "xielu":
+            p, q = torch.nn.functional.softplus(tensors[self.names["act"]].cpu().double()).tolist()
+            self.numbers = (p, 0.5 + q)
 
     def forward(self, x, residual):
-        act = self.up.forward(x, epilogue=self.activation)          # [T,I] in the activation type
-        self.down.forward(act, accumulate_into=residual)
+        """Adds the output into ``residual``, or (``residual`` None) returns it as a new fp32 [T, H]."""
+        act = self.up.forward(x, epilogue=self.activation, numbers=self.numbers)          # [T,I] in the activation type
+        return self.down.forward(act, accumulate_into=residual)
 
 
 class NoFeedForward(Part):

@@ -74,6 +74,7 @@ class PairedRotary(Part):
     and kept as a small fp32 table, the angles and their sines are 32-bit on the device.  It offers no ``encode_and_store``:
     the mixers that use it rotate inside their own prepare step (``kernels.headmix_prepare``) and ask for ``inv_freq``."""
     graph_safe = True
+    halves = False          # how channels are paired: neighbours, or (True) those half the rotated channels apart
 
     def __init__(self, rt, head_dim, rotary_dims=None, theta=10000.0, scaling=None):
         """``scaling`` {"factor", "original", "fast", "slow"} (optional): the pairs that turn fewer than ``slow`` times within
@@ -112,6 +113,7 @@ class PairedRotary(Part):
 class SplitHalfRotary(PairedRotary):
     """The same frequencies, but channel i of the first ``rotary_dims`` channels is paired with channel i + rotary_dims/2
     (the rest pass unchanged).  Like its base it only keeps ``inv_freq``; the mixer's prepare step rotates."""
+    halves = True
 
 
 register_part("position", "rope", RotaryEmbedding, replace=True)

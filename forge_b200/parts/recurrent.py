@@ -22,6 +22,11 @@ The rank of the decay's projection is read from the file's tensors (``rank`` is 
     q_t, k_t rotated by the position (a position part with ``inv_freq``; channel i paired with i + half), k_t times K^-1/2
     S <- g_n S + k_t v_t^T;   o_t = S^T q_t;   every head's o divided by its root mean square (no weight), times silu(Wg h);
     projected back.
+
+"gated_linear" (gated linear attention; N heads of K key and V value channels, state [K, V], no softmax, no denominator):
+    a_t = sigmoid(Wa2 (Wa1 h) + b)^(1/tau)  (a decay per key channel; the hidden layer's size is read from the file)
+    S <- diag(a_t) S + k_t v_t^T;   o_t = K^-1/2 S^T q_t;   every head's o divided by its root mean square, times a weight per value
+    channel that the heads share, times silu(Wg h); projected back.
 """
 import torch
 
@@ -231,6 +236,65 @@ class RetentionMixer(Part):
         return self.o.forward(y, accumulate_into=residual)
 
 
+class GatedLinearMixer(Part):
+    graph_safe = True       # request boundaries and state rows come from the batch's device tensors (q_start, slots)
+
+    def __init__(self, rt, hidden_size, num_heads, head_dim, tau, eps, v_head_dim=None, rank=16, prefix="mix."):
+        if head_dim > 256:
+            raise ConfigError(f"the gated linear mixer takes heads of up to 256 key channels, not {head_dim}")
+        if not tau > 0.0:
+            raise ConfigError(f"the gated linear mixer's decays are a sigmoid to the power 1/tau with a positive tau, not {tau}")
+        self.rt, self.hidden_size, self.num_heads, self.head_dim = rt, hidden_size, num_heads, head_dim
+        self.v_head_dim = head_dim if v_head_dim is None else v_head_dim
+        self.tau, self.eps, self.rank, self.prefix = float(tau), float(eps), int(rank), prefix
+
+    def _n(self, short):
+        return self.prefix + short
+
+    def tensor_specs(self):
+        W, NK, NV = self.hidden_size, self.num_heads * self.head_dim, self.num_heads * self.v_head_dim
+        return {self._n("q"): TensorSpec((NK, W)), self._n("k"): TensorSpec((NK, W)), self._n("v"): TensorSpec((NV, W)),
+                self._n("g"): TensorSpec((NV, W)), self._n("a1"): TensorSpec((-1, W), default_shape=(self.rank, W)),
+                self._n("a2"): TensorSpec((NK, -1), default_shape=(NK, self.rank)), self._n("a2.b"): TensorSpec((NK,), role="bias"),
+                self._n("norm"): TensorSpec((self.v_head_dim,), role="norm"), self._n("o"): TensorSpec((W, NV))}
+
+    def bind(self, tensors):
+        a1, a2 = tensors[self._n("a1")], tensors[self._n("a2")]
+        if a1.shape[0] != a2.shape[1]:
+            from ..weights.loader import WeightError
+            raise WeightError(self._n("a1"), wrong=[f"{self._n('a1')} has {a1.shape[0]} rows, {self._n('a2')} {a2.shape[1]} columns"])
+        self.rank = int(a1.shape[0])
+        # q, k, v, the gate and the decay's hidden layer read the same input: one product
+        self.proj = Linear(self._matrix(torch.cat([tensors[self._n(m)] for m in ("q", "k", "v", "g")] + [a1], dim=0)), None, self.rt)
+        self.a2t = self._vector_f32(a2.t())                          # fp32 [rank, N*K]
+        self.a_bias = self._vector_f32(tensors[self._n("a2.b")])
+        self.norm = self._vector_f32(tensors[self._n("norm")])
+        self.o = Linear(self._matrix(tensors[self._n("o")]), None, self.rt)
+
+    def cache_spec(self):
+        return StateSpec((self.num_heads * self.head_dim * self.v_head_dim,), torch.float32)
+
+    def in_width(self):
+        return 2 * self.num_heads * (self.head_dim + self.v_head_dim) + self.rank
+
+    def out_width(self):
+        return self.num_heads * self.v_head_dim
+
+    def mix(self, p, col, batch, cache, out=None):
+        """p fp32 [T, >= col + in_width]: [q | k | v | g | hidden] from column ``col``; returns the gated heads [T, N*V] (or writes them
+        into ``out`` = (matrix, first column))."""
+        N, K, V = self.num_heads, self.head_dim, self.v_head_dim
+        NK, NV = N * K, N * V
+        o = kernels.gla_scan((p, col), (p, col + NK), (p, col + 2 * NK), (p, col + 2 * NK + 2 * NV), self.rank, self.a2t, self.a_bias, self.tau,
+                             batch, cache.state, N, K, V)
+        return kernels.head_finish(o, self.norm, (p, col + 2 * NK + NV), N, V, self.eps, "silu", self.rt.dtype, out=out)
+
+    def forward(self, x, batch, cache, residual):
+        """Adds the mixer's output into ``residual``, or (``residual`` None) returns it as a new fp32 [T, W]."""
+        return self.o.forward(self.mix(self.proj.forward(x), 0, batch, cache), accumulate_into=residual)
+
+
+register_part("mixer", "gated_linear", GatedLinearMixer, replace=True)
 register_part("mixer", "retention", RetentionMixer, replace=True)
 register_part("mixer", "gated_write", GatedWriteMixer, replace=True)
 register_part("mixer", "wkv", WKVMixer, replace=True)
