@@ -162,7 +162,7 @@ def main():
     ap.add_argument("--no-points", action="store_true", help="skip batch 1 / 64 and the prefill")
     ap.add_argument("--no-shapes", action="store_true", help="skip the Llama-3-8B and Qwen2.5-7B shaped points")
     ap.add_argument("--block-size", type=int, default=64, help="tokens per cache page (named in config)")
-    ap.add_argument("--design", default=None, choices=["zatupel", "tidenex", "tuzavik", "natalorn"],
+    ap.add_argument("--design", default=None, choices=["zatupel", "tidenex", "tuzavik", "natalorn", "ramupel"],
                     help="instead of the default workload: prefill and decode speed of that design at a few layer sizes, "
                          "beside the LLaMA decoder of equal width, depth and head counts")
     a = ap.parse_args()
@@ -694,8 +694,72 @@ class NatalornBench(ShapeBench):
         return flops
 
 
+def ramupel_shape(width, layers, heads, dim, ff, state_heads, state_dim, vocab, **_):
+    """A Ramupel configuration at a real model's layer sizes: latent attention (``heads`` heads of ``dim`` unrotated, dim/2 rotated and
+    ``dim`` value channels over a latent of 4*dim channels), two layers of gated linear attention and a latent attention, in turn; the
+    feed-forward is ungated and half as wide again, so that a token passes through as many of its weights as in the gated ones."""
+    lat = {"type": "latent_attention", "mixer": {"heads": heads, "dim": dim, "rot_dim": dim // 2, "vdim": dim, "kv_rank": 4 * dim,
+                                                 "scale": (dim + dim // 2) ** -0.5, "rot": {"dims": dim // 2, "base": 10000.0}}}
+    gla = {"type": "gla", "mixer": {"heads": state_heads, "dim": state_dim, "vdim": state_dim, "tau": 16.0}}
+    return {"architecture": "Ramupel", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": float(width) ** 0.5},
+            "max_positions": 8192, "layers": [dict(lat if i % 4 in (0, 3) else gla, mlp={"kind": "dense", "ff": 3 * ff // 2}) for i in range(layers)]}
+
+
+RAMUPEL_DECAY_RANK = 16          # the hidden layer of the decays' projection, as random weights draw it
+
+
+def ramupel_matmul_params(cfg):
+    """Matrix elements of all layers, and of the head (the embedding table)."""
+    W, total = cfg.width, 0
+    for layer in cfg.layers:
+        m = layer["mixer"]
+        if layer["type"] == "gla":
+            NK, NV = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+            total += W * (2 * NK + 2 * NV) + W * NV + RAMUPEL_DECAY_RANK * (W + NK)
+        else:
+            H, D, R, E, C = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+            total += W * (H * (D + R) + C + R + H) + H * D * C + H * E * C + W * H * E
+        total += W * W * (2 if layer.get("mlp") else 1)                       # the sublayers' gates
+        if layer.get("mlp"):
+            total += 2 * W * layer["mlp"]["ff"]
+    return total, cfg.vocab * W
+
+
+class RamupelBench(ShapeBench):
+    """ShapeBench's measurements for a Ramupel configuration: only bytes and FLOPs are counted otherwise."""
+
+    def decode_bytes(self, B, ctx):
+        """Every matrix once, and per request the latent rows of every layer that caches some, the state matrices, read and written, and
+        the stream's history: a layer reads what all before it left and writes its own."""
+        cfg = self.cfg
+        layers, head = ramupel_matmul_params(cfg)
+        total = 2 * (layers + head)
+        for i, layer in enumerate(cfg.layers):
+            m = layer["mixer"]
+            if layer["type"] == "gla":
+                total += B * 2 * 4 * m["heads"] * m["dim"] * m["vdim"]
+            else:
+                total += B * ctx * (m["kv_rank"] + m["rot_dim"]) * 2
+            total += B * (i + 2) * cfg.width * 4
+        return total
+
+    def prefill_flops(self, T):
+        """Products, the attention as the design states it (per visible pair and head: scores over dim + rot_dim channels, values of
+        vdim; the engine's absorbed form executes kv_rank + rot_dim and kv_rank instead), 4 FLOPs per state element and token."""
+        cfg = self.cfg
+        layers, head = ramupel_matmul_params(cfg)
+        flops, pairs = 2 * T * layers + 2 * head, T * (T + 1) // 2
+        for layer in cfg.layers:
+            m = layer["mixer"]
+            if layer["type"] == "gla":
+                flops += 4 * T * m["heads"] * m["dim"] * m["vdim"]
+            else:
+                flops += 2 * pairs * m["heads"] * (m["dim"] + m["rot_dim"] + m["vdim"])
+        return flops
+
+
 def design_arm(a):
-    """Prefill and decode speed of the Zatupel, Tidenex, Tuzavik or Natalorn design at a few layer sizes (random weights), each beside the LLaMA decoder
+    """Prefill and decode speed of the Zatupel, Tidenex, Tuzavik, Natalorn or Ramupel design at a few layer sizes (random weights), each beside the LLaMA decoder
     of the same width, depth, head counts and feed-forward width run the same way: decode device-timed at batch 1, 8 and
     64 after 512-token prompts, one prompt step of 2,048 tokens.  One JSON line."""
     import torch
@@ -727,6 +791,8 @@ def design_arm(a):
             arms = [("tuzavik", tuzavik_shape(**z), TuzavikBench), ("tidenex", tidenex_shape(**z), TidenexBench), arms[1]]
         if a.design == "natalorn":        # beside the design whose latent attention and routed experts are its own, and the plain decoder
             arms = [("natalorn", natalorn_shape(**z), NatalornBench), ("tuzavik", tuzavik_shape(**z), TuzavikBench), arms[1]]
+        if a.design == "ramupel":         # beside the design whose latent attention and state scan are the nearest, and the plain decoder
+            arms = [("ramupel", ramupel_shape(**z), RamupelBench), ("tuzavik", tuzavik_shape(**z), TuzavikBench), arms[1]]
         for arch, shape, maker in arms:
             b = maker(shape, PROMPT_LEN, 64, steps, a.warmup, a.block_size, prefill_tokens=PREFILL_TOKENS)
             r = {}

@@ -258,6 +258,16 @@ def case(name):
         mix, ow, iw, wn = torch.eye(S, device=DEV), torch.ones(S, device=DEV) * 0.1, torch.ones(S, device=DEV) * 0.25, torch.ones(W_, device=DEV)
         return (lambda: streams_mix(xs, S, y=y, mix=mix, out_w=ow, in_next=iw, w_next=wn, eps=1e-5, out_dtype=torch.bfloat16)), \
             T * W_ * (2 * S * 4 + 4 + 2), 2 * T * W_ * S * (S + 2)
+    if name in ("depth_step_prefill", "depth_step_decode"):
+        # a stream of 2,048 channels averaged over the depth, the eighth layer's step: two gated outputs join x, the sum over seven older
+        # planes and the new one, the next layer's norm, for 4,096 tokens (508 MB) or 8
+        from forge_b200.kernels import depth_step
+        T, n, W_ = (4096 if name.endswith("prefill") else 8), 8, 2048
+        planes, y1, y2 = torch.randn(n + 2, T, W_, device=DEV), torch.randn(T, W_, device=DEV), torch.randn(T, W_, device=DEV)
+        z, c, wn = torch.randn(T, 2 * W_, device=DEV), torch.rand(n, device=DEV), torch.ones(W_, device=DEV)
+        return (lambda: depth_step(planes, n, n + 1, y1, y2, gates=(z, 0, W_), weights=c, new_plane=n - 1, s_plane=n + 1,
+                                   next_norm=("layer", wn, None, 1e-5), out_dtype=torch.bfloat16)), \
+            T * W_ * (4 * (n - 1 + 1 + 2 + 2 + 2) + 2), T * W_ * (2 * n + 20)
     if name == "routed_pairs_decode":
         # routed experts, one token: 2 of 8 experts of [7168 x 4096] gate, up and down matrices, each (token, expert) pair streaming
         # its expert's rows once (352 MB read, far more than L2 holds); router included
@@ -290,7 +300,19 @@ def case(name):
             kk.copy_(k0)
             retention_scan((qq, 0), (kk, 0), (v, 0), batch, freq, K ** -0.5, decay, state, N, K, K)
         return run, 3 * T * N * K * 4, 4 * T * N * K * K
-    raise SystemExit(f"unknown case {name!r}; known: windowed_attention_prefill chunked_attention_prefill windowed_attention_decode windowed_latent_prefill windowed_latent_decode streams_mix_prefill streams_mix_decode routed_pairs_decode latent_attention_prefill latent_attention_prefill_512 latent_attention_decode retention_scan scored_attention_prefill scored_attention_decode distance_attention_prefill state_scan_gated headmix_attention_prefill headmix_attention_decode state_scan_wkv state_scan_delta "
+    if name == "gla_scan":
+        # gated linear attention's recurrence alone: one request of 1,024 tokens, 32 heads of 64 key and 64 value channels (4 FLOPs per
+        # state element and token), with the kernel that makes the decays from a hidden layer of 16 in front of it
+        from forge_b200.kernels import gla_scan
+        T, N, K, r = 1024, 32, 64, 16
+        mk = lambda n: torch.randn(T, n, device=DEV) * 0.5
+        qq, kk, v, u = mk(N * K), mk(N * K), mk(N * K), mk(r)
+        w2t, b = torch.randn(r, N * K, device=DEV) * 0.3, torch.randn(N * K, device=DEV)
+        state = torch.zeros(2, N * K * K, device=DEV)
+        i32 = lambda z: torch.tensor(z, dtype=torch.int32, device=DEV)
+        batch = SimpleNamespace(q_start=i32([0, T]), slots=i32([1]), num_requests=1)
+        return (lambda: gla_scan((qq, 0), (kk, 0), (v, 0), (u, 0), r, w2t, b, 16.0, batch, state, N, K, K)), 4 * T * N * K * 4, 4 * T * N * K * K
+    raise SystemExit(f"unknown case {name!r}; known: depth_step_prefill depth_step_decode gla_scan windowed_attention_prefill chunked_attention_prefill windowed_attention_decode windowed_latent_prefill windowed_latent_decode streams_mix_prefill streams_mix_decode routed_pairs_decode latent_attention_prefill latent_attention_prefill_512 latent_attention_decode retention_scan scored_attention_prefill scored_attention_decode distance_attention_prefill state_scan_gated headmix_attention_prefill headmix_attention_decode state_scan_wkv state_scan_delta "
                      "gemm_decode_gateup gemm_decode_down gemm_decode_lmhead gemm_prefill_qkv "
                      "gemm_prefill_gateup "
                      "gemm_prefill_qkv_rope gemm_prefill_down attention_decode attention_decode_fused attention_decode_stream attention_prefill "
