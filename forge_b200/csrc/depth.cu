@@ -66,42 +66,37 @@ depth_step_kernel(const DepthStep d, TOut* __restrict__ normed) {
     const P* xp = reinterpret_cast<const P*>(d.planes + (size_t)d.x_plane * d.plane + row);
     const P* y1 = reinterpret_cast<const P*>(d.y1 + row);
     const P* y2 = d.y2 ? reinterpret_cast<const P*>(d.y2 + row) : nullptr;
+    const P* z1 = zr ? reinterpret_cast<const P*>(zr + d.z1) : nullptr;
+    const P* z2 = zr && y2 ? reinterpret_cast<const P*>(zr + d.z2) : nullptr;
     const float* base = d.planes + row;
     const int packs = W / V;
     float sum = 0.f;
     for (int i = threadIdx.x; i < packs; i += blockDim.x) {
-        P x = xp[i], a = y1[i], z{};
-        if (zr) {
-            z = reinterpret_cast<const P*>(zr + d.z1)[i];
+        // all loads ahead of the first store.  The planes that are summed are not written here (x's own may be, by this thread)
+        P x = xp[i], a = __ldg(y1 + i), b{}, ga{}, gb{}, s{};
+        if (y2) b = __ldg(y2 + i);
+        if (z1) ga = __ldg(z1 + i);
+        if (z2) gb = __ldg(z2 + i);
+#pragma unroll 2
+        for (int j = 0; j < d.n - 1; ++j) {
+            P h = __ldg(reinterpret_cast<const P*>(base + (size_t)j * d.plane) + i);
+            const float cj = d.c[j];
 #pragma unroll
-            for (int e = 0; e < V; ++e) lane_of(a, e) *= sigmoidf(lane_of(z, e));
-        }
-        if (y2) {
-            P b = y2[i];
-            if (zr) {
-                z = reinterpret_cast<const P*>(zr + d.z2)[i];
-#pragma unroll
-                for (int e = 0; e < V; ++e) lane_of(b, e) *= sigmoidf(lane_of(z, e));
-            }
-#pragma unroll
-            for (int e = 0; e < V; ++e) lane_of(a, e) += lane_of(b, e);
+            for (int e = 0; e < V; ++e) lane_of(s, e) = fmaf(cj, lane_of(h, e), lane_of(s, e));
         }
 #pragma unroll
-        for (int e = 0; e < V; ++e) lane_of(x, e) += lane_of(a, e);              // X_new
+        for (int e = 0; e < V; ++e) {
+            if (z1) lane_of(a, e) *= sigmoidf(lane_of(ga, e));
+            if (z2) lane_of(b, e) *= sigmoidf(lane_of(gb, e));
+            lane_of(x, e) += y2 ? lane_of(a, e) + lane_of(b, e) : lane_of(a, e);              // X_new
+        }
         if (d.new_plane >= 0) *reinterpret_cast<P*>(d.planes + (size_t)d.new_plane * d.plane + row + (size_t)i * V) = x;
-        P s = x;
         if (d.n > 0) {
-            s = P{};
-#pragma unroll 4
-            for (int j = 0; j < d.n - 1; ++j) {
-                P h = *reinterpret_cast<const P*>(base + (size_t)j * d.plane + (size_t)i * V);
-                const float cj = d.c[j];
-#pragma unroll
-                for (int e = 0; e < V; ++e) lane_of(s, e) = fmaf(cj, lane_of(h, e), lane_of(s, e));
-            }
             const float cn = d.c[d.n - 1];
 #pragma unroll
             for (int e = 0; e < V; ++e) lane_of(s, e) = fmaf(cn, lane_of(x, e), lane_of(s, e));
+        } else {
+            s = x;
         }
         if (d.s_plane >= 0) *reinterpret_cast<P*>(d.planes + (size_t)d.s_plane * d.plane + row + (size_t)i * V) = s;
         if (d.w) {
@@ -149,9 +144,10 @@ cudaError_t run(const DepthStep& d, void* normed, int R, cudaStream_t stream) {
         if (e != cudaSuccess) return e;
         done = true;
     }
-    // few rows: as many threads as the row has packs, so that a row is one trip to memory; many rows: 256 and less
+    // few rows: as many threads as the row has packs, so that a row is one trip to memory; many rows: 128 (5.3 to 5.6 TB/s at rows of
+    // 2,048 and 4,096 channels; 256 threads 4.5 to 5.4, 64 threads 3.4 to 5.6, fewer registers per thread slower at every size)
     int threads = (d.W / V + 31) / 32 * 32;
-    const int most = R <= 148 ? kMaxThreads : 256;
+    const int most = R <= 148 ? kMaxThreads : 128;
     threads = threads < 32 ? 32 : (threads > most ? most : threads);
     return forge::launch(depth_step_kernel<TOut, V>, dim3(R), dim3(threads), smem, stream, 1, d, (TOut*)normed);
 }

@@ -110,3 +110,22 @@ def test_the_fourth_design_option_too():
     per_token, _ = bench.natalorn_matmul_params(cfg)
     assert layers - per_token == 5 * 6 * 3 * 256 * 128                    # six of eight experts of five routed layers
     assert bench._visible_pairs(10, window=4) == 1 + 2 + 3 + 7 * 4 and bench._visible_pairs(10, chunk=4) == 10 + 10 + 3
+
+
+def test_the_fifth_design_option_too():
+    rc, lines = _run("--design", "ramupel", "--gpus", "2")
+    assert rc == 2 and len(lines) == 1 and "single-GPU" in json.loads(lines[0])["error"]
+    sys.path.insert(0, ROOT)
+    import bench
+    import torch
+    from forge_b200.config import config_from_dict
+    from forge_b200.engine.model import Model
+    from forge_b200.parts import Runtime
+    z = dict(width=256, layers=5, heads=8, kv_heads=2, dim=32, ff=512, state_heads=4, state_dim=32, rank=16, window=64, vocab=300)
+    cfg = config_from_dict(bench.ramupel_shape(**z))
+    assert [l["type"] for l in cfg.layers] == ["latent_attention", "gla", "gla", "latent_attention", "latent_attention"]
+    # counted from the configuration alone, the matrices are what the model's own tensor list holds (the head is the embedding)
+    layers, head = bench.ramupel_matmul_params(cfg)
+    specs = Model(cfg.plan(), Runtime(torch.device("cpu"), torch.bfloat16)).tensor_specs()
+    shapes = {n: s.default_shape or s.shape for n, s in specs.items() if s.required and n != "embed"}
+    assert layers == sum(a[0] * a[1] for a in shapes.values() if len(a) == 2) and head == 300 * 256
