@@ -95,12 +95,12 @@ latent_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
 #pragma unroll
     for (int i = 0; i < VC / 8; ++i) oacc[i][0] = oacc[i][1] = oacc[i][2] = oacc[i][3] = 0.f;
     float row_m[2] = {-INFINITY, -INFINITY}, row_l[2] = {0.f, 0.f};
-    // A tile of at most 16 rows would leave three warps idle: there all four warps take the same 16 rows, each computes the
-    // scores again, and each takes a quarter of the chunk's value columns.
+    // A tile of at most 16 (32) rows would leave three (two) warps idle: there all four (two and two) warps take the same 16 rows,
+    // each computes the scores again, and each takes a quarter (a half) of the chunk's value columns.
     const int vcols = min(VC, C - v0);                                    // a multiple of 16
-    const bool colsplit = rows <= 16 && vcols % 64 == 0;
-    const int rb = colsplit ? 0 : warp;                                   // this warp's block of 16 rows
-    const int ntw = colsplit ? vcols / 32 : vcols / 8, cb = colsplit ? warp * (vcols / 4) : 0;     // its value columns: ntw blocks of 8 from cb
+    const int share = rows <= 16 && vcols % 64 == 0 ? 4 : (rows <= 32 && vcols % 32 == 0 ? 2 : 1);     // warps to a block of rows
+    const int rb = warp / share;                                          // this warp's block of 16 rows
+    const int ntw = vcols / 8 / share, cb = (warp % share) * (vcols / share);     // its value columns: ntw blocks of 8 from cb
     const int r_lo = rb * 16 + (lane >> 2), r_hi = r_lo + 8;             // this thread's two rows
     const int pos_lo = pos0 + min(r_lo, rows - 1) / nh, pos_hi = pos0 + min(r_hi, rows - 1) / nh;
     const bool live_lo = r_lo < rows, live_hi = r_hi < rows;
@@ -262,7 +262,7 @@ latent_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
         const int r = h ? r_hi : r_lo;
         if (r >= rows || rb * 16 >= rows) continue;
         const size_t head_index = (size_t)sp * T * H + (size_t)(t0 + r / nh) * H + h0 + r % nh;
-        if (nsplit > 1 && v0 == 0 && (lane & 3) == 0 && (!colsplit || warp == 0)) {
+        if (nsplit > 1 && v0 == 0 && (lane & 3) == 0 && warp % share == 0) {
             part_ml[head_index * 2] = row_m[h];
             part_ml[head_index * 2 + 1] = row_l[h];
         }

@@ -16,6 +16,8 @@
 //   gated linear attention:    S <- diag(a_t) S + k_t v_t^T ;   o_t = K^-1/2 S^T q_t            (a decay per key channel from a
 //                              a_t = sigmoid(W2 u_t + b)^(1/tau)                                 low-rank projection, lowrank_decay_kernel)
 //
+// (a step of single tokens: gla_token_kernel, the whole of it with the head's norm and gate)
+//
 // In the last three the state is [K, V] with V value channels that need not equal K; the first two have V = K.
 //
 // A CTA per (request, head, 16 columns of S) walks the request's tokens of the step in order; column j of S (the K numbers
@@ -391,6 +393,89 @@ lowrank_decay_kernel(ScanInput u, const float* __restrict__ w2t, const float* __
         if (tt < nt) a[(size_t)(t0 + tt) * M + c] = expf((fminf(acc[tt], 0.f) - log1pf(expf(-fabsf(acc[tt])))) * inv_tau);
 }
 
+constexpr int kTokenThreads = 256;
+
+// Gated linear attention where every request of the step brings ONE token: the decays, the state's step, the output, its norm, the
+// weight and the gate in one kernel, a CTA per (request, head).  The state is walked row by row in packs of P value channels
+// (neighbouring threads hold neighbouring packs, so a row is one contiguous read and write); with CG packs a row, thread t holds
+// pack t % CG of the rows t / CG, t / CG + RG, ... and the RG partial outputs of a channel are added in a fixed order.
+template <int P> struct StatePack;
+template <> struct StatePack<1> { using type = float; };
+template <> struct StatePack<4> { using type = float4; };
+__device__ __forceinline__ float& pack_lane(float& v, int) { return v; }
+__device__ __forceinline__ float& pack_lane(float4& v, int i) { return (&v.x)[i]; }
+
+template <int P, typename TA>
+__global__ void __launch_bounds__(kTokenThreads)
+gla_token_kernel(ScanInput q, ScanInput k, ScanInput v, ScanInput g, ScanInput u, int r, const float* __restrict__ w2t, const float* __restrict__ b,
+                 float inv_tau, float q_scale, float* __restrict__ state, long long state_stride, const int32_t* __restrict__ q_start,
+                 const int32_t* __restrict__ slots, const float* __restrict__ weight, float eps, TA* __restrict__ out, long long out_ld,
+                 int N, int K, int V, int CG, int RG) {
+    using S4 = typename StatePack<P>::type;
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float red[32];
+    float* qs = sm;                    // [K]
+    float* ks = qs + K;                // [K]
+    float* as = ks + K;                // [K]
+    float* us = as + K;                // [r]
+    float* os = us + r;                // [RG][V] partial outputs
+    forge::pdl_launch_dependents();
+    forge::pdl_wait();
+    const int s = blockIdx.x, head = blockIdx.y, tid = threadIdx.x;
+    const size_t t = q_start[s];
+    float* S = state + (size_t)slots[s] * state_stride + (size_t)head * K * V;
+    for (int i = tid; i < K; i += kTokenThreads) {
+        qs[i] = q.p[t * q.ld + head * K + i];
+        ks[i] = k.p[t * k.ld + head * K + i];
+    }
+    for (int i = tid; i < r; i += kTokenThreads) us[i] = u.p[t * u.ld + i];
+    __syncthreads();
+    for (int i = tid; i < K; i += kTokenThreads) {
+        const int c = head * K + i, M = N * K;
+        float z = b[c];
+#pragma unroll 8
+        for (int j = 0; j < r; ++j) z = fmaf(us[j], w2t[(size_t)j * M + c], z);
+        as[i] = expf((fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau);
+    }
+    __syncthreads();
+    const int rg = tid / CG, packs = V / P;
+    if (rg < RG) {
+        for (int cp = tid % CG; cp < packs; cp += CG) {
+            S4 vv{}, acc{};
+#pragma unroll
+            for (int e = 0; e < P; ++e) pack_lane(vv, e) = v.p[t * v.ld + (size_t)head * V + cp * P + e];
+#pragma unroll 4
+            for (int row = rg; row < K; row += RG) {
+                S4* ps = reinterpret_cast<S4*>(S + (size_t)row * V) + cp;
+                S4 x = *ps;
+                const float a = as[row], kk = ks[row], qq = qs[row];
+#pragma unroll
+                for (int e = 0; e < P; ++e) {
+                    pack_lane(x, e) = fmaf(a, pack_lane(x, e), kk * pack_lane(vv, e));
+                    pack_lane(acc, e) = fmaf(qq, pack_lane(x, e), pack_lane(acc, e));
+                }
+                *ps = x;
+            }
+#pragma unroll
+            for (int e = 0; e < P; ++e) os[rg * V + cp * P + e] = pack_lane(acc, e);
+        }
+    }
+    __syncthreads();
+    float ss = 0.f;
+    for (int c = tid; c < V; c += kTokenThreads) {
+        float o = 0.f;
+        for (int i = 0; i < RG; ++i) o += os[i * V + c];
+        o *= q_scale;
+        os[c] = o;                      // (row 0 of the partial outputs; nobody else reads column c)
+        ss = fmaf(o, o, ss);
+    }
+    const float inv = 1.0f / sqrtf(forge::block_sum(ss, red) / (float)V + eps);
+    for (int c = tid; c < V; c += kTokenThreads) {
+        const float gv = g.p[t * g.ld + (size_t)head * V + c];
+        out[t * out_ld + (size_t)head * V + c] = forge::from_float<TA>(os[c] * inv * weight[c] * (gv * sigmoidf(gv)));
+    }
+}
+
 template <int MODE, typename TA>
 cudaError_t launch_scan(int kmax, dim3 grid, cudaStream_t stream, ScanInput r, ScanInput k, ScanInput v, ScanInput d, ScanInput a,
                         const float* bonus, const float* inv, float* state, long long stride, const int32_t* q_start, const int32_t* slots,
@@ -519,6 +604,34 @@ extern "C" int forge_gla_scan(const float* q, int ld_q, const float* k, int ld_k
     e = launch_scan<4, float>(kmax, grid, stream, Q, Kk, V, D, D, nullptr, nullptr, state, state_stride, q_start, slots, out, nullptr, 0, 0, N,
                               K, KV, vec, q_scale);
     return forge::check_launch("gla_scan", e);
+}
+
+// The same for a step in which every request brings one token (S tokens, request s's is token q_start[s]), with the head's norm
+// (weight fp32 [KV], eps), and silu of the gate g (fp32 rows, N*KV columns) multiplied on; out of out_dtype, rows of out_ld with the
+// N*KV values at their start.
+extern "C" int forge_gla_token(const float* q, int ld_q, const float* k, int ld_k, const float* v, int ld_v, const float* g, int ld_g,
+                               const float* u, int ld_u, int r, const float* w2t, const float* b, float inv_tau, float q_scale, float* state,
+                               long long state_stride, const int32_t* q_start, const int32_t* slots, const float* weight, float eps, void* out,
+                               int out_dtype, long long out_ld, int S, int N, int K, int KV, cudaStream_t stream) {
+    if (S < 0 || N <= 0 || K <= 0 || KV <= 0 || r <= 0 || ld_u < r || out_ld < (long long)N * KV)
+        return forge::fail(FORGE_ERR_ARG, "gla_token: bad sizes S=%d N=%d K=%d V=%d r=%d", S, N, K, KV, r);
+    if (state_stride < (long long)N * K * KV) return forge::fail(FORGE_ERR_ARG, "gla_token: state rows are too short");
+    if (S == 0) return FORGE_OK;
+    const bool vec = KV % 4 == 0 && state_stride % 4 == 0 && ((long long)K * KV) % 4 == 0 && ((uintptr_t)state & 15) == 0;
+    const int packs = KV / (vec ? 4 : 1), CG = packs < kTokenThreads ? packs : kTokenThreads;
+    int RG = kTokenThreads / CG;
+    if (RG > K) RG = K;
+    const size_t smem = sizeof(float) * ((size_t)3 * K + r + (size_t)RG * KV);
+    if (smem > 48 * 1024) return forge::fail(FORGE_ERR_UNSUPPORTED, "gla_token: heads of %d x %d channels, a hidden layer of %d", K, KV, r);
+    const ScanInput Q{q, ld_q}, Kk{k, ld_k}, V{v, ld_v}, G{g, ld_g}, U{u, ld_u};
+    cudaError_t e = cudaSuccess;
+    FORGE_DISPATCH_DTYPE(out_dtype, TO, {
+        e = vec ? forge::launch(gla_token_kernel<4, TO>, dim3(S, N), dim3(kTokenThreads), smem, stream, 1, Q, Kk, V, G, U, r, w2t, b, inv_tau, q_scale,
+                                state, state_stride, q_start, slots, weight, eps, (TO*)out, out_ld, N, K, KV, CG, RG)
+                : forge::launch(gla_token_kernel<1, TO>, dim3(S, N), dim3(kTokenThreads), smem, stream, 1, Q, Kk, V, G, U, r, w2t, b, inv_tau, q_scale,
+                                state, state_stride, q_start, slots, weight, eps, (TO*)out, out_ld, N, K, KV, CG, RG);
+    });
+    return forge::check_launch("gla_token", e);
 }
 
 // h, out of type dtype: [T, W] and [n_mix, T, W]; mu fp32 [n_mix, W]; the kept row of request s: state + slots[s] * stride + prev_off.

@@ -80,6 +80,7 @@ _SIGNATURES = {
         "forge_head_finish": [_P, _P, _P, _I, _P, _I, _I, _I, _I, _F, _I, _F, _I, _LL, _P],
         "forge_tanh_rows": [_P, _I, _P, _I, _I, _I, _P],
         "forge_gla_scan": [_P, _I] * 4 + [_I, _P, _P, _F, _F, _P, _P, _LL, _P, _P, _P, _I, _I, _I, _I, _I, _P],
+        "forge_gla_token": [_P, _I] * 5 + [_I, _P, _P, _F, _F, _P, _LL, _P, _P, _P, _F, _P, _I, _LL, _I, _I, _I, _I, _P],
         "forge_retention_scan": [_P, _I, _P, _I, _P, _I, _P, _P, _I, _F, _P, _P, _LL, _P, _P, _P, _I, _I, _I, _I, _I, _P],
     },
     "latent": {
@@ -1149,8 +1150,35 @@ def gla_scan(q, k, v, hidden, rank, w2t, bias, tau, batch, state, N, K, KV):
     return out
 
 
+GLA_TOKEN_STATE = 1 << 15           # numbers of a head's state that one CTA walks at most
+
+
+def gla_token_supports(batch, N, K, KV, rank):
+    """A step in which every request brings one token, and heads small enough for one CTA each."""
+    return batch.num_tokens == batch.num_requests and K * KV <= GLA_TOKEN_STATE and 4 * (3 * K + rank + max(KV, 1024)) <= 48 * 1024
+
+
+def gla_token(q, k, v, gate, hidden, rank, w2t, bias, tau, batch, state, N, K, KV, weight, eps, out_dtype, out=None):
+    """``gla_scan`` for a step in which every request brings one token, followed by the head's norm (``weight`` fp32 [KV], eps) and the
+    silu of ``gate`` ((fp32 matrix, first column)): one kernel; returns [T, N*KV] in ``out_dtype`` (or writes them into ``out`` =
+    (matrix, first column))."""
+    lib = library("mixers")
+    T = q[0].shape[0]
+    if T != batch.num_requests or tuple(w2t.shape) != (rank, N * K) or bias.numel() != N * K or weight.numel() != KV or not tau > 0.0:
+        raise KernelError(f"gla_token: {T} tokens of {batch.num_requests} requests, w2 {tuple(w2t.shape)}, {weight.numel()} weights do not fit")
+    out, out_ptr, out_ld = _out_slice(out, N * KV, T, out_dtype, q[0].device)
+    (qp, ql), (kp, kl), (vp, vl), (gp, gl), (up, ul) = _cols(*q), _cols(*k), _cols(*v), _cols(*gate), _cols(*hidden)
+    _check(lib, lib.forge_gla_token(
+        qp, ql, kp, kl, vp, vl, gp, gl, up, ul, int(rank), _need(w2t, "w2t", torch.float32, 2), _need(bias, "bias", torch.float32), 1.0 / float(tau),
+        float(K) ** -0.5, _need(state, "state", torch.float32, 2), state.shape[1], _need(batch.q_start, "q_start", torch.int32),
+        _need(batch.slots, "slots", torch.int32), _need(weight, "weight", torch.float32), float(eps), out_ptr, dtype_code(out_dtype), out_ld,
+        batch.num_requests, N, K, KV, _stream()), "gla_token")
+    return out
+
+
 # ---------------------------------------------------------------------------------------------- latent attention
 
+LATENT_SPLITS = 16                  # runs that a request's rows are dealt out in, at most
 LATENT_KEYS_PER_CHUNK = 32          # fixed: a token's sums must not depend on the step's shape
 
 
@@ -1247,7 +1275,7 @@ def latent_attention(q, cache, group_batch, batch, H, C, R, page_size, scale, wi
             # one CTA per SM, as far as the longest context (the graph's bucket) has tiles
             ctas = T * -(-H // HG) * -(-C // 256)
             reach = min(batch.max_context, window + 63) if window else batch.max_context
-            nsplit = max(1, min(8, -(-reach // 64), _sm_count(q.device) // max(1, ctas)))
+            nsplit = max(1, min(LATENT_SPLITS, -(-reach // 64), _sm_count(q.device) // max(1, ctas)))
         u = new_tensor((nsplit, T, H, C), torch.float32, q.device) if nsplit > 1 else None
         part_ml = new_tensor((nsplit, T, H, 2), torch.float32, q.device) if nsplit > 1 else None
         out = new_tensor((T, H * C), q.dtype, q.device)

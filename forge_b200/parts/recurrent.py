@@ -285,9 +285,12 @@ class GatedLinearMixer(Part):
         into ``out`` = (matrix, first column))."""
         N, K, V = self.num_heads, self.head_dim, self.v_head_dim
         NK, NV = N * K, N * V
-        o = kernels.gla_scan((p, col), (p, col + NK), (p, col + 2 * NK), (p, col + 2 * NK + 2 * NV), self.rank, self.a2t, self.a_bias, self.tau,
-                             batch, cache.state, N, K, V)
-        return kernels.head_finish(o, self.norm, (p, col + 2 * NK + NV), N, V, self.eps, "silu", self.rt.dtype, out=out)
+        q, k, v, g, hidden = (p, col), (p, col + NK), (p, col + 2 * NK), (p, col + 2 * NK + NV), (p, col + 2 * NK + 2 * NV)
+        if kernels.gla_token_supports(batch, N, K, V, self.rank):        # a step of single tokens: one kernel
+            return kernels.gla_token(q, k, v, g, hidden, self.rank, self.a2t, self.a_bias, self.tau, batch, cache.state, N, K, V, self.norm,
+                                     self.eps, self.rt.dtype, out=out)
+        o = kernels.gla_scan(q, k, v, hidden, self.rank, self.a2t, self.a_bias, self.tau, batch, cache.state, N, K, V)
+        return kernels.head_finish(o, self.norm, g, N, V, self.eps, "silu", self.rt.dtype, out=out)
 
     def forward(self, x, batch, cache, residual):
         """Adds the mixer's output into ``residual``, or (``residual`` None) returns it as a new fp32 [T, W]."""

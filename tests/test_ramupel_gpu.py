@@ -144,6 +144,7 @@ GLA = {
     "heads_of_128": dict(num_heads=2, head_dim=128, v_head_dim=64, tau=16.0, rank=8),
     "heads_of_160": dict(num_heads=1, head_dim=160, v_head_dim=24, tau=30.0, rank=16),
     "heads_of_256": dict(num_heads=2, head_dim=256, v_head_dim=20, tau=9.0, rank=1),
+    "a_state_too_large_for_one_cta": dict(num_heads=1, head_dim=256, v_head_dim=144, tau=12.0, rank=4),
     "many_heads": dict(num_heads=20, head_dim=4, v_head_dim=8, tau=2.0, rank=200),
 }
 
@@ -202,6 +203,43 @@ def test_the_state_is_carried_in_32_bits(K, V, r):
         assert max_rel_err(state[slots[s]], S.reshape(-1)) <= 1e-5
     for s in (1, 3):
         assert torch.equal(state[s].cpu(), state0[s])                       # slots that take no part
+
+
+@pytest.mark.parametrize("dtype", DT)
+@pytest.mark.parametrize("K, V, r", [(10, 17, 3), (64, 64, 16), (96, 132, 8), (5, 2, 1), (20, 1100, 40), (256, 128, 2)])
+def test_one_token_of_every_request_in_one_kernel(dtype, K, V, r):
+    """The kernel of single-token steps: what it returns (normed, weighted, gated) and the states it leaves; rows of several
+    requests, slots in any order, inputs that are columns of a wider matrix, an output slice; states whose rows no vector load fits."""
+    from types import SimpleNamespace
+    from forge_b200 import kernels
+    N, B, pad = 3, 4, 5 if V % 2 else 8
+    w2, b, tau, nw = rand(N * K, r, seed=5, scale=0.5), rand(N * K, seed=6) + 1.0, 5.0, 1.0 + rand(V, seed=8, scale=0.3)
+    p = rand(B, pad + 2 * N * (K + V) + r, seed=1)
+    cut = [pad, pad + N * K, pad + 2 * N * K, pad + 2 * N * K + N * V, pad + 2 * N * K + 2 * N * V]
+    q, k, v, g, u = (p[:, c:c + n].double() for c, n in zip(cut, (N * K, N * K, N * V, N * V, r)))
+    state0 = rand(6, N * K * V, seed=7)
+    slots, i32 = [4, 0, 5, 2], lambda z: torch.tensor(z, dtype=torch.int32, device=DEV)
+    batch = SimpleNamespace(q_start=i32([0, 1, 2, 3, 4]), slots=i32(slots), num_requests=B, num_tokens=B)
+    assert kernels.gla_token_supports(batch, N, K, V, r)
+    d, state = lambda z: z.to(DEV).contiguous(), state0.to(DEV)
+    pd = d(p)
+    out = torch.full((B, N * V + 7), 3.0, dtype=dtype, device=DEV)
+    kernels.gla_token(*[(pd, c) for c in cut], r, d(w2.t()), d(b), tau, batch, state, N, K, V, d(nw), 1e-3, dtype, out=(out, 2))
+    a = (torch.sigmoid(u @ w2.double().T + b.double()) ** (1 / tau)).view(B, N, K)
+    for s in range(B):
+        o, S = PR.gated_recurrence(q[s:s + 1].view(1, N, K) * K ** -0.5, k[s:s + 1].view(1, N, K), v[s:s + 1].view(1, N, V), a[s:s + 1],
+                                   state=state0[slots[s]].double().view(N, K, V))
+        want = PR.rms_norm(o, nw.double(), 1e-3).reshape(-1) * g[s] * torch.sigmoid(g[s])
+        assert max_rel_err(out[s, 2:2 + N * V], want) <= PART_TOL[dtype]
+        assert max_rel_err(state[slots[s]], S.reshape(-1)) <= 1e-5
+    for s in (1, 3):
+        assert torch.equal(state[s].cpu(), state0[s])
+    assert bool((out[:, :2] == 3.0).all()) and bool((out[:, 2 + N * V:] == 3.0).all())
+    # portions, and heads too large for one CTA, take the scan
+    batch.num_tokens = B + 1
+    assert not kernels.gla_token_supports(batch, N, K, V, r)
+    batch.num_tokens = B
+    assert not kernels.gla_token_supports(batch, N, 256, 512, r)
 
 
 @pytest.mark.parametrize("dtype", DT)
