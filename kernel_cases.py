@@ -312,7 +312,19 @@ def case(name):
         i32 = lambda z: torch.tensor(z, dtype=torch.int32, device=DEV)
         batch = SimpleNamespace(q_start=i32([0, T]), slots=i32([1]), num_requests=1)
         return (lambda: gla_scan((qq, 0), (kk, 0), (v, 0), (u, 0), r, w2t, b, 16.0, batch, state, N, K, K)), 4 * T * N * K * 4, 4 * T * N * K * K
-    raise SystemExit(f"unknown case {name!r}; known: depth_step_prefill depth_step_decode gla_scan windowed_attention_prefill chunked_attention_prefill windowed_attention_decode windowed_latent_prefill windowed_latent_decode streams_mix_prefill streams_mix_decode routed_pairs_decode latent_attention_prefill latent_attention_prefill_512 latent_attention_decode retention_scan scored_attention_prefill scored_attention_decode distance_attention_prefill state_scan_gated headmix_attention_prefill headmix_attention_decode state_scan_wkv state_scan_delta "
+    if name == "gla_token_decode":
+        # a step of single tokens of 256 requests, 32 heads of 64 x 64: decays, state (read and written once: 268 MB), norm and gate
+        from forge_b200.kernels import gla_token
+        B, N, K, r = 256, 32, 64, 16
+        mk = lambda n: torch.randn(B, n, device=DEV) * 0.5
+        qq, kk, v, g, u = mk(N * K), mk(N * K), mk(N * K), mk(N * K), mk(r)
+        w2t, b, nw = torch.randn(r, N * K, device=DEV) * 0.3, torch.randn(N * K, device=DEV), torch.ones(K, device=DEV)
+        state = torch.zeros(B, N * K * K, device=DEV)
+        i32 = lambda z: torch.tensor(z, dtype=torch.int32, device=DEV)
+        batch = SimpleNamespace(q_start=i32(list(range(B + 1))), slots=i32(list(range(B))), num_requests=B, num_tokens=B)
+        return (lambda: gla_token((qq, 0), (kk, 0), (v, 0), (g, 0), (u, 0), r, w2t, b, 16.0, batch, state, N, K, K, nw, 1e-5, torch.bfloat16)), \
+            B * N * K * (2 * 4 * K + 4 * 4 + 2), 5 * B * N * K * K
+    raise SystemExit(f"unknown case {name!r}; known: depth_step_prefill depth_step_decode gla_scan gla_token_decode windowed_attention_prefill chunked_attention_prefill windowed_attention_decode windowed_latent_prefill windowed_latent_decode streams_mix_prefill streams_mix_decode routed_pairs_decode latent_attention_prefill latent_attention_prefill_512 latent_attention_decode retention_scan scored_attention_prefill scored_attention_decode distance_attention_prefill state_scan_gated headmix_attention_prefill headmix_attention_decode state_scan_wkv state_scan_delta "
                      "gemm_decode_gateup gemm_decode_down gemm_decode_lmhead gemm_prefill_qkv "
                      "gemm_prefill_gateup "
                      "gemm_prefill_qkv_rope gemm_prefill_down attention_decode attention_decode_fused attention_decode_stream attention_prefill "
