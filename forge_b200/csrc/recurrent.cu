@@ -369,12 +369,12 @@ constexpr int kDecayThreads = 128, kDecayTokens = 8;
 __global__ void __launch_bounds__(kDecayThreads)
 lowrank_decay_kernel(ScanInput u, const float* __restrict__ w2t, const float* __restrict__ b, float* __restrict__ a, int T, int r, int M,
                      float inv_tau) {
-    extern __shared__ float us[];                     // [kDecayTokens][r]
+    extern __shared__ __align__(16) float us[];       // [r][kDecayTokens]: the eight tokens' numbers of a hidden channel side by side
     forge::pdl_wait();             // (no early word: the scan follows, see scan_gates_kernel)
     const int t0 = blockIdx.x * kDecayTokens, nt = min(kDecayTokens, T - t0);
     for (int i = threadIdx.x; i < kDecayTokens * r; i += kDecayThreads) {
-        const int tt = i / r;
-        us[i] = tt < nt ? u.p[(size_t)(t0 + tt) * u.ld + i % r] : 0.f;
+        const int tt = i / r, k = i % r;
+        us[k * kDecayTokens + tt] = tt < nt ? u.p[(size_t)(t0 + tt) * u.ld + k] : 0.f;
     }
     __syncthreads();
     const int c = blockIdx.y * kDecayThreads + threadIdx.x;
@@ -385,8 +385,15 @@ lowrank_decay_kernel(ScanInput u, const float* __restrict__ w2t, const float* __
 #pragma unroll 8
     for (int k = 0; k < r; ++k) {
         const float w = w2t[(size_t)k * M + c];
+        const float4* u4 = reinterpret_cast<const float4*>(us + k * kDecayTokens);
 #pragma unroll
-        for (int tt = 0; tt < kDecayTokens; ++tt) acc[tt] = fmaf(us[tt * r + k], w, acc[tt]);
+        for (int h = 0; h < kDecayTokens / 4; ++h) {
+            const float4 x = u4[h];
+            acc[4 * h] = fmaf(x.x, w, acc[4 * h]);
+            acc[4 * h + 1] = fmaf(x.y, w, acc[4 * h + 1]);
+            acc[4 * h + 2] = fmaf(x.z, w, acc[4 * h + 2]);
+            acc[4 * h + 3] = fmaf(x.w, w, acc[4 * h + 3]);
+        }
     }
 #pragma unroll
     for (int tt = 0; tt < kDecayTokens; ++tt)
