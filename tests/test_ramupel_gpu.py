@@ -635,6 +635,7 @@ def test_generation_through_the_scheduler(ram, dtype):
     out = model.generate(prompt, max_new_tokens=12, do_sample=False)
     assert out["num_generated_tokens"] == 12 and out["finish_reason"] == "length"
     logits_fn = lambda ids: plain.forward(ids).float()
+    assert len(set(out["token_ids"])) >= 4                                   # a text that repeats one token would show little
     assert_greedy_follows_plain(logits_fn, prompt, out["token_ids"], TOL[dtype], what="generate")
     sched = forge.RequestScheduler(model, max_num_seqs=2, max_tokens_per_step=48)
     prompts = [reqs["r0"][:50], reqs["r2"][:9], reqs["r3"][:31], reqs["r1"][:3]]
