@@ -5,6 +5,7 @@ from .tidenex import TidenexConfig
 from .tuzavik import TuzavikConfig
 from .natalorn import NatalornConfig
 from .ramupel import RamupelConfig
+from .zuretar import ZuretarConfig
 from .registry import (config_from_dict, load_config, register_architecture, registered_architectures,
                        unregister_architecture)
 
@@ -31,5 +32,9 @@ register_architecture("Natalorn", NatalornConfig, replace=True)
 # one cached latent per token with a gate per head, or gated linear attention; ungated feed-forwards
 register_architecture("Ramupel", RamupelConfig, replace=True)
 
-__all__ = ["ZatupelConfig", "TidenexConfig", "TuzavikConfig", "NatalornConfig", "RamupelConfig", "ConfigError", "LayerSpec", "ModelPlan", "PartSpec", "LlamaConfig", "config_from_dict", "load_config",
+# parallel layers with one norm, some of which use another layer's weights: a gated delta rule behind short convolutions, or chunked
+# attention beside lightning attention with normed outputs; dense or routed feed-forwards
+register_architecture("Zuretar", ZuretarConfig, replace=True)
+
+__all__ = ["ZatupelConfig", "TidenexConfig", "TuzavikConfig", "NatalornConfig", "RamupelConfig", "ZuretarConfig", "ConfigError", "LayerSpec", "ModelPlan", "PartSpec", "LlamaConfig", "config_from_dict", "load_config",
            "register_architecture", "registered_architectures", "unregister_architecture"]

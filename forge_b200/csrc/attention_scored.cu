@@ -9,10 +9,12 @@
 //   window      position i sees j only if i - j < window                              (0: no such limit)
 //   chunk       position i sees j only if i / chunk == j / chunk (integer division)     (0: no such limit)
 //   softcap     score <- softcap tanh(score / softcap), after the scale                (0: none)
+//   sink        the softmax denominator of head h also counts exp(sink_h), which has no key and no value   (null: none; M = 1)
 //
 // and in the prepare step:  an RMS norm over ALL of a token's query channels (and all of its key channels) with a
 // weight per channel; a query temperature 1 + coef ln(floor((p + 1) / every) + 1) at position p; a rotation of the first
-// rot_dims channels of every map, channel i paired with i + rot_dims/2.
+// rot_dims channels of every map, channel i paired with i + rot_dims/2.  A second prepare step (M = 1, scored_prepare_heads_kernel) rotates
+// with cos and sin multiplied by a number, and then divides every query and key head by its root mean square.
 //
 // Query heads have M*D channels, key heads M*D, value heads E; a cache page is [kv head][token in page][M*D] keys followed
 // by [kv head][token in page][E] values.  All arithmetic is fp32 whatever the storage type.  Keys are walked in chunks of KT
@@ -88,6 +90,76 @@ scored_prepare_kernel(const float* __restrict__ proj, int ld, const int32_t* __r
             vbase[((size_t)(idx / E) * page_size + off) * E + idx % E] = forge::from_float<TC>(row[QW + KW + idx]);
 }
 
+constexpr int kHeadRegs = 8;           // rotated pairs, and twice as many channels that pass, that a lane holds of a head at most
+
+// One warp per (token, head): the QU query heads, the KU key heads (both D channels) and the KU value heads (E channels) of fp32 row
+// [q | k | v].  A query or key head's first rot_dims channels turn by position * inv_freq (channel i with i + rot_dims/2; cos and sin
+// times amp), then (norm) the head is divided by its root mean square.  Queries go to q_out, keys and values to their cache rows.
+template <typename TC>
+__global__ void __launch_bounds__(kPrepThreads)
+scored_prepare_heads_kernel(const float* __restrict__ proj, int ld, const int32_t* __restrict__ positions,
+                            const int32_t* __restrict__ slot_mapping, const float* __restrict__ inv_freq, float amp, TC* __restrict__ q_out,
+                            TC* __restrict__ cache, int QU, int KU, int D, int E, int rot_dims, int norm, float eps, int page_size,
+                            long long page_stride) {
+    forge::pdl_launch_dependents();
+    forge::pdl_wait();
+    const int t = blockIdx.x, lane = threadIdx.x & 31, unit = blockIdx.y * (kPrepThreads / 32) + (threadIdx.x >> 5);
+    if (unit >= QU + 2 * KU) return;
+    const int slot = slot_mapping ? slot_mapping[t] : -1;
+    const bool store = slot >= 0 && FORGE_SLOT_OK(slot);
+    const int page = store ? slot / page_size : 0, off = store ? slot % page_size : 0;
+    TC* kbase = cache + (size_t)page * page_stride;
+    if (unit >= QU + KU) {                     // a value head passes as it is
+        if (!store) return;
+        const int g = unit - QU - KU;
+        const float* v = proj + (size_t)t * ld + (size_t)(QU + KU) * D + (size_t)g * E;
+        TC* dst = kbase + (size_t)KU * page_size * D + ((size_t)g * page_size + off) * E;
+        for (int c = lane; c < E; c += 32) dst[c] = forge::from_float<TC>(v[c]);
+        return;
+    }
+    if (unit >= QU && !store) return;
+    const float* x = proj + (size_t)t * ld + (size_t)unit * D;
+    TC* dst = unit < QU ? q_out + ((size_t)t * QU + unit) * D : kbase + ((size_t)(unit - QU) * page_size + off) * D;
+    const int half = rot_dims >> 1;
+    const float pos = (float)positions[t];
+    float lo[kHeadRegs], hi[kHeadRegs], pass[2 * kHeadRegs], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < kHeadRegs; ++i) {
+        const int c = lane + 32 * i;
+        lo[i] = hi[i] = 0.f;
+        if (c < half) {
+            float s, cs;
+            sincosf(pos * inv_freq[c], &s, &cs);
+            s *= amp;
+            cs *= amp;
+            const float u = x[c], v = x[c + half];
+            lo[i] = u * cs - v * s;
+            hi[i] = v * cs + u * s;
+            ss = fmaf(lo[i], lo[i], fmaf(hi[i], hi[i], ss));
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < 2 * kHeadRegs; ++i) {
+        const int c = rot_dims + lane + 32 * i;
+        pass[i] = c < D ? x[c] : 0.f;
+        ss = fmaf(pass[i], pass[i], ss);
+    }
+    const float inv = norm ? 1.0f / sqrtf(forge::warp_sum(ss) / (float)D + eps) : 1.0f;
+#pragma unroll
+    for (int i = 0; i < kHeadRegs; ++i) {
+        const int c = lane + 32 * i;
+        if (c < half) {
+            dst[c] = forge::from_float<TC>(lo[i] * inv);
+            dst[c + half] = forge::from_float<TC>(hi[i] * inv);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < 2 * kHeadRegs; ++i) {
+        const int c = rot_dims + lane + 32 * i;
+        if (c < D) dst[c] = forge::from_float<TC>(pass[i] * inv);
+    }
+}
+
 constexpr int kAttThreads = 256;
 
 // The first position that position `pos` sees.  It does not fall as pos grows.
@@ -107,7 +179,7 @@ scored_attention_kernel(const TC* __restrict__ q, const TC* __restrict__ cache, 
                         const int32_t* __restrict__ tile_t0, const int32_t* __restrict__ tile_n, const float* __restrict__ r1,
                         const float* __restrict__ r2, TC* __restrict__ out, int H, int G, int M, int D, int E, int page_size,
                         long long page_stride, int max_pages, float scale, float lambda, float post, float eps, float out_scale,
-                        int TQ, int KT, long long out_ld, int window, int chunk, float softcap) {
+                        int TQ, int KT, long long out_ld, int window, int chunk, float softcap, const float* __restrict__ sink) {
     extern __shared__ float smem[];
     forge::pdl_launch_dependents();
     forge::pdl_wait();
@@ -215,7 +287,13 @@ scored_attention_kernel(const TC* __restrict__ q, const TC* __restrict__ cache, 
     if (M == 1) {
         for (int i = tid; i < rows * E; i += kAttThreads) {
             const int e = i % E, row = i / E, r = row % R, tq = row / R;
-            out[(size_t)(t0 + tq) * out_ld + (size_t)(g * R + r) * E + e] = forge::from_float<TC>(acc[i] / ls[row] * out_scale);
+            float a = acc[i], l = ls[row];
+            if (sink) {
+                const float b = sink[g * R + r], m = fmaxf(ms[row], b), x = expf(ms[row] - m);
+                a *= x;
+                l = l * x + expf(b - m);
+            }
+            out[(size_t)(t0 + tq) * out_ld + (size_t)(g * R + r) * E + e] = forge::from_float<TC>(a / l * out_scale);
         }
         return;
     }
@@ -270,6 +348,30 @@ extern "C" int forge_scored_prepare(const float* proj, int ld, const int32_t* po
     return forge::check_launch("scored_prepare", e);
 }
 
+// The prepare step that works head by head: proj fp32 [T, ld], per row QU query heads of D channels, KU key heads of D, KU value heads
+// of E.  inv_freq fp32 [rot_dims / 2] (null with rot_dims 0), amp: what cos and sin are multiplied by; norm: every query and key head is
+// divided by its root mean square after the rotation.  cache: pages of page_stride elements; slot_mapping null: nothing stored.
+extern "C" int forge_scored_prepare_heads(const float* proj, int ld, const int32_t* positions, const int32_t* slot_mapping,
+                                          const float* inv_freq, float amp, void* q_out, void* cache, int dtype, int T, int QU, int KU, int D,
+                                          int E, int rot_dims, int norm, float eps, int page_size, long long page_stride, cudaStream_t stream) {
+    if (T < 0 || QU <= 0 || KU <= 0 || D <= 0 || E <= 0 || page_size <= 0 || rot_dims < 0 || rot_dims > D || (rot_dims & 1))
+        return forge::fail(FORGE_ERR_ARG, "scored_prepare_heads: bad sizes T=%d QU=%d KU=%d D=%d E=%d rot=%d page=%d", T, QU, KU, D, E, rot_dims,
+                           page_size);
+    if (D > 64 * kHeadRegs) return forge::fail(FORGE_ERR_UNSUPPORTED, "scored_prepare_heads: heads of %d channels", D);
+    if (rot_dims > 0 && !inv_freq) return forge::fail(FORGE_ERR_ARG, "scored_prepare_heads: a rotation needs its frequencies");
+    if (ld < (QU + KU) * D + KU * E) return forge::fail(FORGE_ERR_ARG, "scored_prepare_heads: rows of %d are too short", ld);
+    if (slot_mapping && (!cache || page_stride < (long long)page_size * KU * (D + E)))
+        return forge::fail(FORGE_ERR_ARG, "scored_prepare_heads: pages are too small");
+    if (T == 0) return FORGE_OK;
+    const int units = QU + 2 * KU, warps = kPrepThreads / 32;
+    cudaError_t e = cudaSuccess;
+    FORGE_DISPATCH_DTYPE(dtype, TT,
+        e = forge::launch(scored_prepare_heads_kernel<TT>, dim3(T, (units + warps - 1) / warps), dim3(kPrepThreads), 0, stream, 1, proj, ld,
+                          positions, slot_mapping, inv_freq, amp, (TT*)q_out, (TT*)cache, QU, KU, D, E, rot_dims, norm, eps, page_size,
+                          page_stride));
+    return forge::check_launch("scored_prepare_heads", e);
+}
+
 // Bytes of shared memory of a tile of TQ tokens with key chunks of KT (the caller picks TQ with it).
 extern "C" long long forge_scored_attention_smem(int H, int G, int M, int D, int E, int TQ, int KT) {
     return (long long)scored_smem_bytes(H / (G > 0 ? G : 1), M, D, E, TQ, KT);
@@ -277,12 +379,13 @@ extern "C" long long forge_scored_attention_smem(int H, int G, int M, int D, int
 
 // q [T, H*M*D] and out (rows of out_ld elements, the heads' H*E values at their start) in the cache's type.  tile_t0 / tile_n int32 [num_tiles] (both null: one token a tile).
 // r1, r2 fp32 [H] or both null.  M = 2: lambda, post and eps of the combination of the two maps.  window, chunk, softcap: 0 = none.
+// sink fp32 [H] or null (M = 1 only).
 extern "C" int forge_scored_attention(const void* q, const void* cache, const int32_t* block_table, const int32_t* tok_req,
                                       const int32_t* positions, const int32_t* tile_t0, const int32_t* tile_n, const float* r1,
                                       const float* r2, void* out, int dtype, int num_tiles, int H, int G, int M, int D, int E,
                                       int page_size, long long page_stride, int max_pages, float scale, float lambda, float post,
                                       float eps, float out_scale, int TQ, int KT, long long out_ld, int window, int chunk, float softcap,
-                                      cudaStream_t stream) {
+                                      const float* sink, cudaStream_t stream) {
     if (out_ld < (long long)H * E) return forge::fail(FORGE_ERR_ARG, "scored_attention: output rows of %lld are too short", out_ld);
     if (num_tiles < 0 || H <= 0 || G <= 0 || D <= 0 || E <= 0 || H % G != 0 || (M != 1 && M != 2) || page_size <= 0 || max_pages <= 0 ||
         TQ <= 0 || KT <= 0)
@@ -291,6 +394,7 @@ extern "C" int forge_scored_attention(const void* q, const void* cache, const in
     if ((tile_t0 == nullptr) != (tile_n == nullptr)) return forge::fail(FORGE_ERR_ARG, "scored_attention: half a tile list");
     if ((r1 == nullptr) != (r2 == nullptr)) return forge::fail(FORGE_ERR_ARG, "scored_attention: r1 and r2 go together");
     if (window < 0 || chunk < 0 || softcap < 0.f) return forge::fail(FORGE_ERR_ARG, "scored_attention: window %d, chunk %d, softcap %g", window, chunk, (double)softcap);
+    if (sink && M != 1) return forge::fail(FORGE_ERR_ARG, "scored_attention: a sink beside two maps");
     if (num_tiles == 0) return FORGE_OK;
     const size_t smem = scored_smem_bytes(H / G, M, D, E, TQ, KT);
     if (smem > 200 * 1024)
@@ -305,7 +409,7 @@ extern "C" int forge_scored_attention(const void* q, const void* cache, const in
         }
         e = forge::launch(scored_attention_kernel<TT>, dim3(num_tiles, G), dim3(kAttThreads), smem, stream, 1, (const TT*)q,
                           (const TT*)cache, block_table, tok_req, positions, tile_t0, tile_n, r1, r2, (TT*)out, H, G, M, D, E, page_size,
-                          page_stride, max_pages, scale, lambda, post, eps, out_scale, TQ, KT, out_ld, window, chunk, softcap);
+                          page_stride, max_pages, scale, lambda, post, eps, out_scale, TQ, KT, out_ld, window, chunk, softcap, sink);
     });
     return forge::check_launch("scored_attention", e);
 }

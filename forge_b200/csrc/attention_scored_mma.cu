@@ -72,7 +72,7 @@ scored_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
                   const int32_t* __restrict__ tok_req, const int32_t* __restrict__ positions, const int32_t* __restrict__ tile_t0,
                   const int32_t* __restrict__ tile_n, const float* __restrict__ r1, const float* __restrict__ r2, float* __restrict__ u,
                   __nv_bfloat16* __restrict__ out, float* __restrict__ part_ml, int nsplit_given, int T, int qrows, int H, int G, int M, int D, int E, int page_size, long long page_stride,
-                  int max_pages, float scale, float out_scale, long long out_ld, int window, int chunk, float softcap) {
+                  int max_pages, float scale, float out_scale, long long out_ld, int window, int chunk, float softcap, const float* __restrict__ sink) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     forge::pdl_launch_dependents();
     forge::pdl_wait();
@@ -281,7 +281,14 @@ scored_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
         }
         __syncthreads();                                                  // before a later fetch writes into this buffer
     }
-    const float inv[2] = {nsplit > 1 ? 1.0f : (row_l[0] > 0.f ? 1.0f / row_l[0] : 0.f), nsplit > 1 ? 1.0f : (row_l[1] > 0.f ? 1.0f / row_l[1] : 0.f)};
+    float inv[2] = {nsplit > 1 ? 1.0f : (row_l[0] > 0.f ? 1.0f / row_l[0] : 0.f), nsplit > 1 ? 1.0f : (row_l[1] > 0.f ? 1.0f / row_l[1] : 0.f)};
+    if (sink && nsplit == 1) {           // the denominator also counts the sink (with runs the second kernel adds it, once)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            const float b = sink[h ? h_hi : h_lo] * kLog2e, m = fmaxf(row_m[h], b), x = ex2(row_m[h] - m);
+            inv[h] = x / fmaf(row_l[h], x, ex2(b - m));
+        }
+    }
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
         const int r = h ? r_hi : r_lo;
@@ -310,7 +317,7 @@ scored_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
 // out bf16 [T, H, E].
 __global__ void __launch_bounds__(128)
 scored_combine_kernel(const float* __restrict__ u, const float* __restrict__ part_ml, int nsplit, __nv_bfloat16* __restrict__ out_base, int rows,
-                      int H, int M, int E, float lambda, float post, float eps, long long out_ld) {
+                      int H, int M, int E, float lambda, float post, float eps, long long out_ld, const float* __restrict__ sink) {
     constexpr int kMaxSplit = 16;
     forge::pdl_launch_dependents();
     forge::pdl_wait();
@@ -327,6 +334,11 @@ scored_combine_kernel(const float* __restrict__ u, const float* __restrict__ par
             const float x = l > 0.f ? exp2f(part_ml[at] - mx) : 0.f;          // a run that saw no key counts for nothing
             wt[m][s] = x;
             den = fmaf(x, l, den);
+        }
+        if (sink) {                      // counts once, beside the runs (both in units of log2 e)
+            const float b = sink[w % H] * 1.4426950408889634f, top = fmaxf(mx, b), x = exp2f(mx - top);
+            den = fmaf(den, x, exp2f(b - top));
+            for (int s = 0; s < nsplit; ++s) wt[m][s] *= x;
         }
         const float inv = den > 0.f ? 1.0f / den : 0.f;
         for (int s = 0; s < nsplit; ++s) wt[m][s] *= inv;
@@ -377,7 +389,7 @@ int launch_scored(int which, dim3 grid, size_t smem, cudaStream_t stream, const 
                   const int32_t* bt, const int32_t* tok_req, const int32_t* positions, const int32_t* t0, const int32_t* tn, const float* r1,
                   const float* r2, float* u, __nv_bfloat16* out, float* part_ml, int nsplit, int T, int qrows, int H, int G, int M, int D, int E,
                   int page_size, long long page_stride, int max_pages, float scale, float out_scale, long long out_ld, int window, int chunk,
-                  float softcap) {
+                  float softcap, const float* sink) {
     bool& done = g_attr_done[which + (SPLIT ? 3 : 0)].current();
     if (!done) {
         cudaError_t e = cudaFuncSetAttribute(scored_mma_kernel<VC, SPLIT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMmaSmemLimit);
@@ -387,7 +399,7 @@ int launch_scored(int which, dim3 grid, size_t smem, cudaStream_t stream, const 
     return forge::check_launch("scored_attention_mma",
                                forge::launch(scored_mma_kernel<VC, SPLIT>, grid, dim3(kThreads), smem, stream, 1, q, cache, bt, tok_req, positions, t0,
                                              tn, r1, r2, u, out, part_ml, nsplit, T, qrows, H, G, M, D, E, page_size, page_stride, max_pages, scale,
-                                             out_scale, out_ld, window, chunk, softcap));
+                                             out_scale, out_ld, window, chunk, softcap, sink));
 }
 
 }  // namespace
@@ -403,18 +415,18 @@ extern "C" int forge_scored_mma_supports(int H, int G, int M, int D, int E, int 
 // [nsplit, T, H, M, 2] (scratch, nsplit > 1: steps of single tokens only); out bf16, rows of out_ld elements (even) with the
 // heads' H*E values at their start.  tile_t0 / tile_n: tiles of consecutive
 // tokens of one request with tile_n * (H/G) <= 64 (both null: one token per tile, num_tiles = T).  r1, r2 fp32 [H] or null.
-// window, chunk, softcap: the limits on what a position sees and the cap on the scores, 0 = none.
+// window, chunk, softcap: the limits on what a position sees and the cap on the scores, 0 = none.  sink fp32 [H] or null (M == 1 only).
 extern "C" int forge_scored_attention_mma(const void* q, const void* cache, const int32_t* block_table, const int32_t* tok_req,
                                           const int32_t* positions, const int32_t* tile_t0, const int32_t* tile_n, const float* r1,
                                           const float* r2, float* u, float* part_ml, int nsplit, void* out, int T, int num_tiles, int H, int G, int M, int D, int E,
                                           int page_size, long long page_stride, int max_pages, float scale, float lambda, float post,
                                           float eps, float out_scale, long long out_ld, int window, int chunk, float softcap,
-                                          cudaStream_t stream) {
+                                          const float* sink, cudaStream_t stream) {
     if (out_ld < (long long)H * E || (out_ld & 1)) return forge::fail(FORGE_ERR_ARG, "scored_attention_mma: output rows of %lld elements", out_ld);
     if (!forge_scored_mma_supports(H, G, M, D, E, page_size))
         return forge::fail(FORGE_ERR_UNSUPPORTED, "scored_attention_mma: H=%d G=%d M=%d D=%d E=%d", H, G, M, D, E);
     if (T < 0 || num_tiles < 0 || max_pages <= 0 || (tile_t0 == nullptr) != (tile_n == nullptr) || (r1 == nullptr) != (r2 == nullptr) ||
-        ((M == 2 || nsplit > 1) && !u) || window < 0 || chunk < 0 || softcap < 0.f)
+        ((M == 2 || nsplit > 1) && !u) || (sink && M != 1) || window < 0 || chunk < 0 || softcap < 0.f)
         return forge::fail(FORGE_ERR_ARG, "scored_attention_mma: bad arguments");
     if (nsplit < 1 || nsplit > 16 || (nsplit > 1 && (tile_t0 != nullptr || part_ml == nullptr)))
         return forge::fail(FORGE_ERR_ARG, "scored_attention_mma: the keys are dealt out to several CTAs only in steps of single tokens");
@@ -432,7 +444,7 @@ extern "C" int forge_scored_attention_mma(const void* q, const void* cache, cons
     __nv_bfloat16* ob = (__nv_bfloat16*)out;
     const float os = (M == 1 && nsplit == 1) ? out_scale : 1.0f;
     int rc;
-#define FORGE_SCORED_ARGS grid, smem, stream, qb, cb, block_table, tok_req, positions, tile_t0, tile_n, r1, r2, u, ob, part_ml, nsplit, T, qrows, H, G, M, D, E, page_size, page_stride, max_pages, scale, os, out_ld, window, chunk, softcap
+#define FORGE_SCORED_ARGS grid, smem, stream, qb, cb, block_table, tok_req, positions, tile_t0, tile_n, r1, r2, u, ob, part_ml, nsplit, T, qrows, H, G, M, D, E, page_size, page_stride, max_pages, scale, os, out_ld, window, chunk, softcap, sink
     if (nsplit > 1) rc = VC == 64 ? launch_scored<64, true>(0, FORGE_SCORED_ARGS) : VC == 128 ? launch_scored<128, true>(1, FORGE_SCORED_ARGS) : launch_scored<256, true>(2, FORGE_SCORED_ARGS);
     else rc = VC == 64 ? launch_scored<64, false>(0, FORGE_SCORED_ARGS) : VC == 128 ? launch_scored<128, false>(1, FORGE_SCORED_ARGS) : launch_scored<256, false>(2, FORGE_SCORED_ARGS);
 #undef FORGE_SCORED_ARGS
@@ -440,7 +452,7 @@ extern "C" int forge_scored_attention_mma(const void* q, const void* cache, cons
     const unsigned blocks = (unsigned)(((size_t)T * H + 3) / 4);
     return forge::check_launch("scored_combine", forge::launch(scored_combine_kernel, dim3(blocks), dim3(128), 0, stream, 1, (const float*)u,
                                                                (const float*)part_ml, nsplit, ob, T * H, H, M, E, lambda,
-                                                               (M == 1 ? 1.0f : post) * out_scale, eps, out_ld));
+                                                               (M == 1 ? 1.0f : post) * out_scale, eps, out_ld, sink));
 }
 
 FORGE_DEFINE_CHECKS_ENTRY(attention_scored_mma)

@@ -195,6 +195,7 @@ class Model:
         else:
             residual = self.embedding.forward(batch.token_ids, status=batch.status)
         S = self.plan.streams
+        hands_on = S != 1 or depth or any(getattr(b, "hands_on", False) for b in self.blocks)
         if S != 1:
             residual = kernels.streams_expand(residual, S)          # every copy of the stream starts as the embedding output
         if self._fused_decode_applies(batch):
@@ -214,8 +215,8 @@ class Model:
                 if replay is not None:
                     replay.run(self._replay_tensors[pos] + [position_caches[pos].kv])
                     continue
-                if S != 1 or depth:
-                    # a block may leave the next block's first input in the same pass as its own last write to the copies
+                if hands_on:
+                    # a block may leave the next block's first input in the same pass as its own last write to the stream
                     batch.shared["following_block"] = self.blocks[self.plan.schedule[pos + 1]] if pos + 1 < len(self.plan.schedule) else None
                 if depth:
                     # ... and the last one the head's input: the model's norm of the wanted rows

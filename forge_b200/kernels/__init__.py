@@ -41,6 +41,7 @@ _SIGNATURES = {
         "forge_act_rows": [_P, _I, _P, _I, _I, _I, _I, _F, _F, _P],
         "forge_depth_step": [_P, _LL, _I, _I, _I, _I] + [_P] * 4 + [_I, _I, _I, _P, _P, _I, _F, _P, _I, _P, _I, _I, _P],
         "forge_rmsnorm": [_P, _P, _P, _I, _P, _I, _I, _F, _P],
+        "forge_join": [_P, _I] + [_P, _P, _F] * 4 + [_F, _P, _F, _P, _I, _I, _I, _P],
         "forge_rmsnorm_pair": [_P, _P, _P, _P, _P, _I, _I, _I, _F, _P],
         "forge_rope_kv_write": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _P, _P],
         "forge_rope_table": [_P, _P, _I, _I, _F, _I, _P],
@@ -73,14 +74,22 @@ _SIGNATURES = {
         "forge_headmix_attention_mma": [_P] * 11 + [_I, _P] + [_I] * 7 + [_LL, _I, _I, _I, _F, _P],
         "forge_state_scan": [_I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _P, _P, _P, _LL, _P, _P, _P, _P, _I, _I, _LL, _I, _I, _I, _I, _I, _P],
         "forge_scored_prepare": [_P, _I] + [_P] * 7 + [_I] * 8 + [_F, _F, _F, _I, _LL, _P],
-        "forge_scored_attention": [_P] * 10 + [_I] * 8 + [_LL, _I] + [_F] * 5 + [_I, _I, _LL, _I, _I, _F, _P],
+        "forge_scored_prepare_heads": [_P, _I, _P, _P, _P, _F, _P, _P] + [_I] * 8 + [_F, _I, _LL, _P],
+        "forge_scored_attention": [_P] * 10 + [_I] * 8 + [_LL, _I] + [_F] * 5 + [_I, _I, _LL, _I, _I, _F, _P, _P],
         "forge_scored_mma_supports": [_I] * 6,
-        "forge_scored_attention_mma": [_P] * 11 + [_I, _P] + [_I] * 8 + [_LL, _I] + [_F] * 5 + [_LL, _I, _I, _F, _P],
+        "forge_scored_attention_mma": [_P] * 11 + [_I, _P] + [_I] * 8 + [_LL, _I] + [_F] * 5 + [_LL, _I, _I, _F, _P, _P],
         "forge_token_shift": [_P, _P, _LL, _LL, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P],
         "forge_head_finish": [_P, _P, _P, _I, _P, _I, _I, _I, _I, _F, _I, _F, _I, _LL, _P],
         "forge_tanh_rows": [_P, _I, _P, _I, _I, _I, _P],
         "forge_gla_scan": [_P, _I] * 4 + [_I, _P, _P, _F, _F, _P, _P, _LL, _P, _P, _P, _I, _I, _I, _I, _I, _P],
         "forge_gla_token": [_P, _I] * 5 + [_I, _P, _P, _F, _F, _P, _LL, _P, _P, _P, _F, _P, _I, _LL, _I, _I, _I, _I, _P],
+        "forge_lightning_scan": [_P, _I, _P, _P, _LL, _P, _P, _P] + [_I] * 5 + [_P],
+        "forge_lightning_token": [_P, _I, _P, _P, _LL, _P, _P, _P] + [_I] * 4 + [_P],
+        "forge_gated_delta_scan": [_P, _I] * 3 + [_P, _P, _P, _LL, _P, _P, _P] + [_I] * 6 + [_P],
+        "forge_delta_prepare": [_P, _I, _I, _I, _P, _I, _P, _LL, _LL] + [_P] * 9 + [_I] * 6 + [_P],
+        "forge_gated_delta_token": [_P, _I, _I, _I, _I, _P, _I, _P, _LL, _LL] + [_P] * 6 + [_F, _P, _I, _LL] + [_I] * 5 + [_P],
+        "forge_token_state_supports": [_I] * 3,
+        "forge_gated_rows": [_P, _P, _P, _I, _P, _I, _LL, _I, _I, _F, _P],
         "forge_retention_scan": [_P, _I, _P, _I, _P, _I, _P, _P, _I, _F, _P, _P, _LL, _P, _P, _P, _I, _I, _I, _I, _I, _P],
     },
     "latent": {
@@ -92,7 +101,7 @@ _SIGNATURES = {
         "forge_latent_attention_mma": [_P] * 9 + [_I, _P] + [_I] * 7 + [_F, _I, _P, _P],
     },
     "moe": {
-        "forge_moe_route": [_P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _I, _I, _F, _P],
+        "forge_moe_route": [_P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _I, _I, _I, _F, _P],
         "forge_moe_pair_gate_up": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _LL, _P],
         "forge_moe_pair_down": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P],
         "forge_moe_expert_supports": [_I, _I, _I],
@@ -706,6 +715,29 @@ def depth_step(planes, n, x_plane, y1, y2=None, gates=None, weights=None, new_pl
     return out
 
 
+def join(residual, terms, eps, next_norm=None, out_dtype=None, out=None):
+    """residual fp32 [T, W] += the sum of ``terms``, one to four of (y fp32 [T, W], weight fp32 [W] or None, scale): scale * y, or with a
+    weight scale * y / rms(y) * weight (``eps`` inside the root).  ``next_norm`` = (weight fp32 [W], eps): also returns the new
+    residual / rms * weight in ``out_dtype`` (written into ``out`` if given), else None."""
+    lib = library("core")
+    T, W = residual.shape
+    if not 1 <= len(terms) <= 4 or any(tuple(y.shape) != (T, W) or (w is not None and w.numel() != W) for y, w, _ in terms):
+        raise KernelError(f"join: {len(terms)} terms of {[tuple(y.shape) for y, _, _ in terms]} do not fit a stream of {(T, W)}")
+    args = []
+    for y, w, s in list(terms) + [(None, None, 0.0)] * (4 - len(terms)):
+        args += [_opt(y, "y", torch.float32), _opt(w, "w", torch.float32), float(s)]
+    w_next, eps_next = next_norm if next_norm is not None else (None, 0.0)
+    if w_next is None:
+        out = None
+    else:
+        out = new_tensor((T, W), out_dtype, residual.device) if out is None else out
+        if tuple(out.shape) != (T, W) or w_next.numel() != W:
+            raise KernelError(f"join: the next norm's output {tuple(out.shape)} and weight of {w_next.numel()} do not fit a stream of {(T, W)}")
+    _check(lib, lib.forge_join(_need(residual, "residual", torch.float32, 2), len(terms), *args, float(eps), _opt(w_next, "next_w", torch.float32),
+                               float(eps_next), _opt(out, "out", out_dtype), dtype_code(out_dtype) if out is not None else F32, T, W, _stream()), "join")
+    return out
+
+
 def rmsnorm_pair(x, w1, w2, eps, out_dtype):
     """(x * rsqrt(mean(x^2)+eps) * w1, the same * w2) over the rows of float32 x [T,H]: one read, one reduction."""
     lib = library("core")
@@ -1028,16 +1060,40 @@ def scored_prepare(proj, positions, slot_mapping, cache, H, G, M, D, E, page_siz
     return q
 
 
+def scored_prepare_heads(proj, positions, slot_mapping, cache, H, G, D, E, page_size, act_dtype, inv_freq=None, amp=1.0, norm=False, eps=0.0, col=0):
+    """``scored_prepare`` head by head: every query and key head's first 2*len(inv_freq) channels turn by position * inv_freq (channel i
+    with i + half; cos and sin times ``amp``), then with ``norm`` the head is divided by its root mean square (``eps`` inside the root)."""
+    lib = library("mixers")
+    T, ld = proj.shape
+    if ld - col < (H + G) * D + G * E:
+        raise KernelError(f"scored_prepare_heads: rows of {ld} from column {col} are too short")
+    if cache is not None and cache.dtype != act_dtype:
+        raise KernelError("scored_prepare_heads: cache and activation dtypes differ")
+    q = new_tensor((T, H * D), act_dtype, proj.device)
+    if cache is None:
+        slot_mapping = None
+    stride = _page_stride(cache) if cache is not None else G * page_size * (D + E)
+    rot = 0 if inv_freq is None else 2 * inv_freq.numel()
+    _check(lib, lib.forge_scored_prepare_heads(
+        _need(proj, "proj", torch.float32, 2) + 4 * int(col), ld, _need(positions, "positions", torch.int32), _opt(slot_mapping, "slot_mapping", torch.int32),
+        _opt(inv_freq, "inv_freq", torch.float32) if rot else None, float(amp), _need(q, "q", act_dtype), _opt(cache, "cache"), dtype_code(act_dtype),
+        T, H, G, D, E, rot, 1 if norm else 0, float(eps), page_size, stride, _stream()), "scored_prepare_heads")
+    return q
+
+
 def scored_attention(q, cache, group_batch, batch, H, G, M, D, E, page_size, scale, r1=None, r2=None, lam=0.0, post=1.0, eps=0.0,
-                     out_scale=1.0, out=None, window=0, chunk=0, softcap=0.0):
+                     out_scale=1.0, out=None, window=0, chunk=0, softcap=0.0, sink=None):
     """Causal softmax attention of every token of the step over its request's pages, M maps per head (see
     csrc/attention_scored.cu): scores scale q.k - r1_h ln(1 + r2_h (i - j)); with M = 2 the maps' outputs are combined as
     a1 - lam a2, divided by their root mean square (``eps`` inside the root) and multiplied by ``post``.  Returns [T, H*E] in
     q's type, times ``out_scale``; ``out`` = (matrix, first column): written there instead (the matrix is returned).
     ``window``: key j counts for query i only if i - window < j; ``chunk``: only if i // chunk == j // chunk; ``softcap``: scores
-    become softcap tanh(score / softcap); 0 switches each off."""
+    become softcap tanh(score / softcap); 0 switches each off.  ``sink`` fp32 [H] (M = 1): the softmax denominator of head h also counts
+    exp(sink[h])."""
     lib = library("mixers")
     window, chunk, softcap = int(window or 0), int(chunk or 0), float(softcap or 0.0)
+    if sink is not None and sink.numel() != H:
+        raise KernelError(f"scored_attention: {sink.numel()} sinks for {H} heads")
     T = q.shape[0]
     out, out_ptr, out_ld = _out_slice(out, H * E, T, q.dtype, q.device)
     if q.dtype == torch.bfloat16 and _TENSOR_CORE_ATTENTION and lib.forge_scored_mma_supports.fn(H, G, M, D, E, page_size):
@@ -1057,7 +1113,8 @@ def scored_attention(q, cache, group_batch, batch, H, G, M, D, E, page_size, sca
             _need(batch.tok_req, "tok_req", torch.int32), _need(batch.positions, "positions", torch.int32), _opt(t0, "tile_t0", torch.int32),
             _opt(tn, "tile_n", torch.int32), _opt(r1, "r1", torch.float32), _opt(r2, "r2", torch.float32), _opt(u, "u", torch.float32),
             _opt(part_ml, "part_ml", torch.float32), nsplit, out_ptr, T, tiles, H, G, M, D, E, page_size, _page_stride(cache), group_batch.block_table.shape[1],
-            float(scale), float(lam), float(post), float(eps), float(out_scale), out_ld, window, chunk, softcap, _stream()), "scored_attention_mma")
+            float(scale), float(lam), float(post), float(eps), float(out_scale), out_ld, window, chunk, softcap, _opt(sink, "sink", torch.float32), _stream()),
+            "scored_attention_mma")
         if M == 2 or nsplit > 1:
             count_launches(1)      # the kernel that puts the runs of key tiles, and the two maps, together
         return out
@@ -1071,7 +1128,8 @@ def scored_attention(q, cache, group_batch, batch, H, G, M, D, E, page_size, sca
         _need(batch.tok_req, "tok_req", torch.int32), _need(batch.positions, "positions", torch.int32), _opt(t0, "tile_t0", torch.int32),
         _opt(tn, "tile_n", torch.int32), _opt(r1, "r1", torch.float32), _opt(r2, "r2", torch.float32), out_ptr,
         dtype_code(q.dtype), tiles, H, G, M, D, E, page_size, _page_stride(cache), group_batch.block_table.shape[1], float(scale),
-        float(lam), float(post), float(eps), float(out_scale), TQ, SCORED_KEYS_PER_CHUNK, out_ld, window, chunk, softcap, _stream()), "scored_attention")
+        float(lam), float(post), float(eps), float(out_scale), TQ, SCORED_KEYS_PER_CHUNK, out_ld, window, chunk, softcap,
+        _opt(sink, "sink", torch.float32), _stream()), "scored_attention")
     return out
 
 
@@ -1173,6 +1231,117 @@ def gla_token(q, k, v, gate, hidden, rank, w2t, bias, tau, batch, state, N, K, K
         float(K) ** -0.5, _need(state, "state", torch.float32, 2), state.shape[1], _need(batch.q_start, "q_start", torch.int32),
         _need(batch.slots, "slots", torch.int32), _need(weight, "weight", torch.float32), float(eps), out_ptr, dtype_code(out_dtype), out_ld,
         batch.num_requests, N, K, KV, _stream()), "gla_token")
+    return out
+
+
+# a recurrence whose inputs pass silu, or a short convolution and silu, first (csrc/recurrent_token.cu)
+
+def token_state_supports(batch, K, V, delta):
+    """A step in which every request brings one token, and heads of K x V numbers that the kernel of single tokens takes."""
+    return batch.num_tokens == batch.num_requests and bool(library("mixers").forge_token_state_supports.fn(int(K), int(V), 1 if delta else 0))
+
+
+def lightning_scan(proj, col, decay, batch, state, N, K, V):
+    """proj fp32 [T, >= col + N*(2K+V)]: [q | k | v] from column ``col``, which pass silu IN PLACE; S <- decay[n] S + k v^T, o = S^T q over the
+    step's tokens, request by request, from and into ``state`` fp32 [slots, >= N*K*V].  Returns fp32 [T, N*V]."""
+    lib = library("mixers")
+    T = proj.shape[0]
+    out = new_tensor((T, N * V), torch.float32, proj.device)
+    p, ld = _cols(proj, col)
+    _check(lib, lib.forge_lightning_scan(p, ld, _need(decay, "decay", torch.float32), _need(state, "state", torch.float32, 2), state.shape[1],
+                                         _need(batch.q_start, "q_start", torch.int32), _need(batch.slots, "slots", torch.int32),
+                                         _need(out, "out", torch.float32), T, batch.num_requests, N, K, V, _stream()), "lightning_scan")
+    count_launches(1)              # the kernel that applies silu
+    return out
+
+
+def lightning_token(proj, col, decay, batch, state, N, K, V):
+    """``lightning_scan`` for a step in which every request brings one token (proj is left as it is)."""
+    lib = library("mixers")
+    T = proj.shape[0]
+    if T != batch.num_requests:
+        raise KernelError(f"lightning_token: {T} tokens of {batch.num_requests} requests")
+    out = new_tensor((T, N * V), torch.float32, proj.device)
+    p, ld = _cols(proj, col)
+    _check(lib, lib.forge_lightning_token(p, ld, _need(decay, "decay", torch.float32), _need(state, "state", torch.float32, 2), state.shape[1],
+                                          _need(batch.q_start, "q_start", torch.int32), _need(batch.slots, "slots", torch.int32),
+                                          _need(out, "out", torch.float32), T, N, K, V, _stream()), "lightning_token")
+    return out
+
+
+def gated_rows(o, weight, gate, eps, out_dtype, out=None):
+    """o fp32 [T, n] / rms(o over the row) * ``weight`` fp32 [n] * sigmoid of ``gate`` ((fp32 matrix, first column)), [T, n] in ``out_dtype``
+    (or written into ``out`` = (matrix, first column), the matrix returned)."""
+    lib = library("mixers")
+    T, n = o.shape
+    if weight.numel() != n:
+        raise KernelError(f"gated_rows: {weight.numel()} weights for rows of {n}")
+    out, out_ptr, out_ld = _out_slice(out, n, T, out_dtype, o.device)
+    gp, gl = _cols(*gate)
+    _check(lib, lib.forge_gated_rows(_need(o, "o", torch.float32, 2), _need(weight, "weight", torch.float32), gp, gl, out_ptr, dtype_code(out_dtype),
+                                     out_ld, T, n, float(eps), _stream()), "gated_rows")
+    return out
+
+
+def _delta_state(conv_w, state, N, M, K, V):
+    """(taps, first number of the ring in a state row) of the gated delta rule's state; checks the sizes."""
+    C, taps = 2 * M * K + N * V, conv_w.shape[1]
+    ring_off = N * K * V
+    if conv_w.shape[0] != C or state.shape[1] < ring_off + taps * C:
+        raise KernelError(f"gated delta rule: convolutions {tuple(conv_w.shape)} and state rows of {state.shape[1]} do not fit {N}/{M} heads of {K} x {V}")
+    return taps, ring_off
+
+
+def gated_delta_prepare(proj, col, b_col, a_col, conv_w, decay_rate, dt, batch, state, N, M, K, V):
+    """proj fp32 [T, ..]: [q: M*K | k: M*K | v: N*V] from column ``col``, and from ``b_col`` and ``a_col`` on the N inputs each of the write
+    strengths and the decays.  Convolves q, k, v over time (``conv_w`` fp32 [2*M*K + N*V, taps]; earlier inputs from the ring in the
+    request's ``state`` row behind its N*K*V numbers, which is brought up to date), silu, q and k to unit vectors, q times K^-1/2.
+    Returns (qkv fp32 [T, 2*M*K + N*V], decays fp32 [T, N], strengths fp32 [T, N])."""
+    lib = library("mixers")
+    T = proj.shape[0]
+    taps, ring_off = _delta_state(conv_w, state, N, M, K, V)
+    qkv = new_tensor((T, 2 * M * K + N * V), torch.float32, proj.device)
+    g, beta = new_tensor((T, N), torch.float32, proj.device), new_tensor((T, N), torch.float32, proj.device)
+    p, ld = _cols(proj, col)
+    _check(lib, lib.forge_delta_prepare(
+        p, ld, int(b_col - col), int(a_col - col), _need(conv_w, "conv_w", torch.float32, 2), taps, _need(state, "state", torch.float32, 2), state.shape[1],
+        ring_off, _need(batch.tok_req, "tok_req", torch.int32), _need(batch.q_start, "q_start", torch.int32),
+        _need(batch.positions, "positions", torch.int32), _need(batch.slots, "slots", torch.int32), _need(decay_rate, "decay_rate", torch.float32),
+        _need(dt, "dt", torch.float32), _need(qkv, "qkv"), _need(g, "g"), _need(beta, "beta"), T, batch.num_requests, N, M, K, V, _stream()),
+        "gated_delta_prepare")
+    count_launches(1)              # the kernel that brings the rings up to date
+    return qkv, g, beta
+
+
+def gated_delta_scan(qkv, g, beta, batch, state, N, M, K, V):
+    """The gated delta rule over the step's tokens, request by request, from and into ``state``: per head n with q and k of head n // (N/M),
+    S <- g S;  S <- S + k (beta (v - S^T k))^T;  o = S^T q.  The inputs as ``gated_delta_prepare`` leaves them; returns fp32 [T, N*V]."""
+    lib = library("mixers")
+    T = qkv.shape[0]
+    out = new_tensor((T, N * V), torch.float32, qkv.device)
+    (qp, ld), (kp, _), (vp, _) = _cols(qkv, 0), _cols(qkv, M * K), _cols(qkv, 2 * M * K)
+    _check(lib, lib.forge_gated_delta_scan(
+        qp, ld, kp, ld, vp, ld, _need(g, "g", torch.float32, 2), _need(beta, "beta", torch.float32, 2), _need(state, "state", torch.float32, 2),
+        state.shape[1], _need(batch.q_start, "q_start", torch.int32), _need(batch.slots, "slots", torch.int32), _need(out, "out", torch.float32),
+        T, batch.num_requests, N, M, K, V, _stream()), "gated_delta_scan")
+    return out
+
+
+def gated_delta_token(proj, col, g_col, b_col, a_col, conv_w, decay_rate, dt, batch, state, N, M, K, V, weight, eps, out_dtype, out=None):
+    """Both of the above, the heads' norm (``weight`` fp32 [V], eps) and silu of the gate (N*V columns from ``g_col``) for a step in which every
+    request brings one token: one kernel; returns [T, N*V] in ``out_dtype`` (or writes them into ``out`` = (matrix, first column))."""
+    lib = library("mixers")
+    T = proj.shape[0]
+    if T != batch.num_requests or weight.numel() != V:
+        raise KernelError(f"gated_delta_token: {T} tokens of {batch.num_requests} requests, {weight.numel()} norm weights for {V} channels")
+    taps, ring_off = _delta_state(conv_w, state, N, M, K, V)
+    out, out_ptr, out_ld = _out_slice(out, N * V, T, out_dtype, proj.device)
+    p, ld = _cols(proj, col)
+    _check(lib, lib.forge_gated_delta_token(
+        p, ld, int(g_col - col), int(b_col - col), int(a_col - col), _need(conv_w, "conv_w", torch.float32, 2), taps, _need(state, "state", torch.float32, 2),
+        state.shape[1], ring_off, _need(batch.q_start, "q_start", torch.int32), _need(batch.positions, "positions", torch.int32),
+        _need(batch.slots, "slots", torch.int32), _need(decay_rate, "decay_rate", torch.float32), _need(dt, "dt", torch.float32),
+        _need(weight, "weight", torch.float32), float(eps), out_ptr, dtype_code(out_dtype), out_ld, T, N, M, K, V, _stream()), "gated_delta_token")
     return out
 
 
@@ -1303,12 +1472,12 @@ def latent_attention(q, cache, group_batch, batch, H, C, R, page_size, scale, wi
 
 # ---------------------------------------------------------------------------------------------- routed experts
 
-def moe_route(x, router, top, softmax=False, renorm=False, correction=None, groups=0, keep=0, factor=1.0):
+def moe_route(x, router, top, softmax=False, renorm=False, correction=None, groups=0, keep=0, factor=1.0, group_top=1):
     """(int32 [T, top] experts, fp32 [T, top] weights): the ``top`` largest of sigmoid (or softmax) of router . x per token, the lower
     index winning a tie; the weights are those scores, divided by their sum with ``renorm``, times ``factor``.  router fp32 [E, W];
     fp32 arithmetic.  ``correction`` fp32 [E]: experts are ranked by score + correction (the weights stay the scores).  ``groups``
-    > 1: the experts are cut into that many consecutive blocks of equal size, a block is ranked by the largest ranking number in it,
-    and only the ``keep`` best blocks' experts take part in the ranking."""
+    > 1: the experts are cut into that many consecutive blocks of equal size, a block is ranked by the largest ranking number in it
+    (``group_top`` 2: by the sum of its two largest), and only the ``keep`` best blocks' experts take part in the ranking."""
     lib = library("moe")
     T, W = x.shape
     E = router.shape[0]
@@ -1316,7 +1485,8 @@ def moe_route(x, router, top, softmax=False, renorm=False, correction=None, grou
     wts = new_tensor((T, top), torch.float32, x.device)
     _check(lib, lib.forge_moe_route(_need(x, "x", ndim=2), dtype_code(x.dtype), _need(router, "router", torch.float32, 2), _need(idx, "idx"),
                                     _need(wts, "wts"), T, W, E, int(top), 1 if softmax else 0, 1 if renorm else 0,
-                                    _opt(correction, "correction", torch.float32), int(groups or 0), int(keep or 0), float(factor), _stream()), "moe_route")
+                                    _opt(correction, "correction", torch.float32), int(groups or 0), int(keep or 0), int(group_top), float(factor),
+                                    _stream()), "moe_route")
     return idx, wts
 
 

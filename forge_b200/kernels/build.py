@@ -20,9 +20,9 @@ CSRC = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))),
 
 LIBRARIES = {
     # embedding, norm, rotary + cache write, activation, fp32 GEMM, fp32/any-shape attention, sampling
-    # ... and a residual stream kept as several copies, or averaged over the depth
+    # ... and a residual stream kept as several copies, or averaged over the depth, or to which several normed outputs are added
     "core": ["embedding.cu", "norm.cu", "rope_cache.cu", "activation.cu", "gemm_simt.cu",
-             "attention_simt.cu", "sampling.cu", "streams.cu", "depth.cu"],
+             "attention_simt.cu", "sampling.cu", "streams.cu", "depth.cu", "join.cu"],
     # bf16 tcgen05 + TMA GEMM with fused epilogues
     "gemm_sm100": ["gemm_sm100.cu"],
     # bf16 tensor-core paged attention (mma.sync) for any head size, prompt portions and decode
@@ -32,7 +32,8 @@ LIBRARIES = {
     "attention_sm100": ["attention_sm100.cu"],
     # attention whose heads exchange weights, over a window with kept first tokens; attention with shaped scores (two maps per
     # head, a distance term); mixers with a matrix of state per head
-    "mixers": ["attention_headmix.cu", "attention_headmix_mma.cu", "attention_scored.cu", "attention_scored_mma.cu", "recurrent.cu"],
+    "mixers": ["attention_headmix.cu", "attention_headmix_mma.cu", "attention_scored.cu", "attention_scored_mma.cu", "recurrent.cu",
+               "recurrent_token.cu"],
     # attention over one latent row per token shared by all heads (keys and values per head are never formed), and the
     # per-head products around it
     "latent": ["attention_latent.cu", "attention_latent_mma.cu"],

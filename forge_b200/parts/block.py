@@ -16,6 +16,9 @@ model says which block runs next (``batch.shared["following_block"]``), a layer'
 channel, and what goes on is a weighted sum over the depth, x <- sum_j c[j] X_j of everything the layers have left so far (X_0: the
 embedding output).  The two gates ride in the mixer's input product; the gated sum, the average and the next layer's norm (after
 the last layer the model's norm, on the wanted rows) are one kernel.
+"parallel_one_norm":  r += mixer(h) + feed_forward(h), h = norm(r), one RMS norm whose output both sublayers read.  What a sublayer hands on
+as terms (a routed feed-forward's sum, mixers whose outputs are normed first) joins the stream in one kernel, which also leaves the
+next layer's h; what is the result of a plain product is added in that product's epilogue.
 """
 from ..weights.loader import TensorSpec  # noqa: F401  (re-exported for part authors)
 from .base import Part, build_part, register_part
@@ -365,6 +368,62 @@ class ParallelDepthBlock(Part):
             kernels.depth_step(residual, n, x_plane, y1, y2, **step)
 
 
+class ParallelOneNormBlock(Part):
+    """``norms``: {"input": spec}, an RMS norm."""
+    graph_safe = True
+    hands_on = True          # may leave the next block's first input: the model says which block that is
+
+    def sub_parts(self):
+        return [self.mixer, self.feed_forward, self.norm]
+
+    def __init__(self, rt, layer_spec):
+        from ..config.base import ConfigError
+        from .feedforward import NoFeedForward
+        from .norm import RMSNorm
+        self.rt = rt
+        self.mixer = build_part("mixer", layer_spec.mixer, rt)
+        self.feed_forward = build_part("feed_forward", layer_spec.feed_forward, rt)
+        self.norm = build_part("norm", layer_spec.norms["input"], rt)
+        if type(self.norm) is not RMSNorm:
+            raise ConfigError("a parallel layer with one norm has an RMS norm")
+        self.has_ff = type(self.feed_forward) is not NoFeedForward
+
+    def tensor_specs(self):
+        specs = {}
+        for part in self.sub_parts():
+            specs.update(part.tensor_specs())
+        return specs
+
+    def bind(self, tensors):
+        for part in self.sub_parts():
+            part.bind({name: tensors[name] for name in part.tensor_specs() if name in tensors})
+
+    def forward(self, residual, batch, cache):
+        from .. import kernels
+        T, W = residual.shape
+        left = batch.shared.pop("stream_input", None)          # (the block it is meant for, its input) from the layer before
+        h = left[1] if left is not None and left[0] is self else self.norm.forward(residual)
+        terms, eps = [], 1.0                                    # (eps: of the normed terms)
+        if getattr(self.mixer, "norms", None) is not None and hasattr(self.mixer, "terms"):
+            terms, eps = self.mixer.terms(h, batch, cache), self.mixer.eps
+        else:
+            self.mixer.forward(h, batch, cache, residual)
+        if self.has_ff:
+            if getattr(self.feed_forward, "adds_in_product", True):
+                self.feed_forward.forward(h, residual)
+            else:
+                terms = terms + [(self.feed_forward.forward(h, None), None, 1.0)]
+        if not terms:
+            return
+        nxt = batch.shared.get("following_block")
+        if isinstance(nxt, ParallelOneNormBlock) and nxt.rt.dtype == self.rt.dtype:
+            x = kernels.join(residual, terms, eps, next_norm=(nxt.norm.weight, nxt.norm.eps), out_dtype=self.rt.dtype,
+                             out=step_buffer(batch, T, W, self.rt.dtype, residual.device))
+            batch.shared["stream_input"] = (nxt, x)
+        else:
+            kernels.join(residual, terms, eps)
+
+
 def step_buffer(batch, T, W, dtype, device):
     """One of two [T, W] buffers that live as long as the step, taken in turn: what a layer leaves for the next one."""
     from .. import kernels
@@ -390,3 +449,4 @@ register_part("block", "parallel", ParallelBlock, replace=True)
 register_part("block", "sandwich", SandwichBlock, replace=True)
 register_part("block", "hyper_connections", HyperConnectionBlock, replace=True)
 register_part("block", "parallel_depth", ParallelDepthBlock, replace=True)
+register_part("block", "parallel_one_norm", ParallelOneNormBlock, replace=True)

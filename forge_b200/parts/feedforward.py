@@ -16,23 +16,31 @@ class SwiGLU(Part):
     graph_safe = True
     activation = "swiglu"          # the name of the product's gated epilogue
 
-    def __init__(self, rt, hidden_size, intermediate_size, names=None, suffix=".weight"):
+    def __init__(self, rt, hidden_size, intermediate_size, names=None, suffix=".weight", bias=False):
         """``names``: the three matrices' tensor names without ``suffix`` (a design whose files say "mlp.gate" gives
-        suffix "")."""
+        suffix ""); ``bias``: all three products have biases, named like the matrices with ".b"."""
+        self.bias = bool(bias)
         self.rt, self.hidden_size, self.intermediate_size = rt, hidden_size, intermediate_size
         self.names = {k: v + suffix for k, v in {**DEFAULT_NAMES, **(names or {})}.items()}
         self.gate_up = self.down = None
 
     def tensor_specs(self):
         n, H, I = self.names, self.hidden_size, self.intermediate_size
-        return {n["gate"]: TensorSpec((I, H)), n["up"]: TensorSpec((I, H)), n["down"]: TensorSpec((H, I))}
+        specs = {n["gate"]: TensorSpec((I, H)), n["up"]: TensorSpec((I, H)), n["down"]: TensorSpec((H, I))}
+        if self.bias:
+            specs.update({n[m] + ".b": TensorSpec((rows,), role="bias") for m, rows in (("gate", I), ("up", I), ("down", H))})
+        return specs
 
     def bind(self, tensors):
         n = self.names
         g, u = tensors[n["gate"]], tensors[n["up"]]
         gu = torch.stack([g, u], dim=1).reshape(2 * self.intermediate_size, self.hidden_size)
-        self.gate_up = Linear(self._matrix(gu), None, self.rt)
-        self.down = Linear(self._matrix(tensors[n["down"]]), None, self.rt)
+        b_gu = b_down = None
+        if self.bias:
+            b_gu = self._vector_f32(torch.stack([tensors[n["gate"] + ".b"], tensors[n["up"] + ".b"]], dim=1).reshape(-1))
+            b_down = self._vector_f32(tensors[n["down"] + ".b"])
+        self.gate_up = Linear(self._matrix(gu), b_gu, self.rt)
+        self.down = Linear(self._matrix(tensors[n["down"]]), b_down, self.rt)
 
     def replay_tensors(self):
         return self.gate_up.replay_tensors() + self.down.replay_tensors() if type(self) is SwiGLU else None

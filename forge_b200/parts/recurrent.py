@@ -27,6 +27,16 @@ The rank of the decay's projection is read from the file's tensors (``rank`` is 
     a_t = sigmoid(Wa2 (Wa1 h) + b)^(1/tau)  (a decay per key channel; the hidden layer's size is read from the file)
     S <- diag(a_t) S + k_t v_t^T;   o_t = K^-1/2 S^T q_t;   every head's o divided by its root mean square, times a weight per value
     channel that the heads share, times silu(Wg h); projected back.
+
+"gated_delta" (gated delta rule; N heads of K key and V value channels, state [K, V]; groups of heads share one q and k):
+    q, k, v each pass a short causal convolution over time (a filter per channel) and silu; q and k become unit vectors per head, q times K^-1/2
+    g_t = exp(-exp(A) softplus(Wa h + dt)),  beta_t = sigmoid(Wb h)  (one of each per head)
+    S <- g_t S;   S <- S + k_t (beta_t (v_t - S^T k_t))^T;   o_t = S^T q_t;   every head's o divided by its root mean square, times a weight
+    per value channel that the heads share, times silu(Wg h); projected back.  The convolutions' last inputs are state too.
+
+"lightning" (linear attention with one fixed decay per head; N heads of K key and V value channels, state [K, V]):
+    q, k, v = silu(Wq h), silu(Wk h), silu(Wv h);   S <- g_n S + k_t v_t^T;   o_t = S^T q_t;   all of a token's heads together divided by their
+    root mean square, times a weight per channel, times sigmoid(Wg h); projected back.
 """
 import torch
 
@@ -297,6 +307,133 @@ class GatedLinearMixer(Part):
         return self.o.forward(self.mix(self.proj.forward(x), 0, batch, cache), accumulate_into=residual)
 
 
+class GatedDeltaMixer(Part):
+    graph_safe = True       # positions, request boundaries and state rows come from the batch's device tensors
+    ROW_MULTIPLE = 8        # the projection's rows are filled up to a multiple of this: aligned rows of its result
+
+    def __init__(self, rt, hidden_size, num_heads, head_dim, taps, eps, num_qk_heads=None, v_head_dim=None, prefix="mix."):
+        """``num_qk_heads``: heads of q and k, each shared by num_heads / num_qk_heads neighbouring heads; ``taps``: tokens that the
+        convolutions look at (the current one and taps - 1 before it)."""
+        num_qk_heads = num_heads if num_qk_heads is None else num_qk_heads
+        if head_dim > 256:
+            raise ConfigError(f"the gated delta mixer takes heads of up to 256 key channels, not {head_dim}")
+        if num_qk_heads < 1 or num_heads % num_qk_heads:
+            raise ConfigError(f"gated delta rule: {num_heads} heads cannot share {num_qk_heads} query/key heads")
+        if taps < 1:
+            raise ConfigError(f"gated delta rule: a convolution over {taps} tokens")
+        self.rt, self.hidden_size, self.num_heads, self.num_qk_heads, self.head_dim = rt, hidden_size, num_heads, num_qk_heads, head_dim
+        self.v_head_dim = head_dim if v_head_dim is None else v_head_dim
+        self.taps, self.eps, self.prefix = int(taps), float(eps), prefix
+
+    def _n(self, short):
+        return self.prefix + short
+
+    def _conv_channels(self):
+        return 2 * self.num_qk_heads * self.head_dim + self.num_heads * self.v_head_dim
+
+    def tensor_specs(self):
+        W, N, QK, NV = self.hidden_size, self.num_heads, self.num_qk_heads * self.head_dim, self.num_heads * self.v_head_dim
+        specs = {}
+        for m, rows in (("q", QK), ("k", QK), ("v", NV)):
+            specs.update({self._n(m): TensorSpec((rows, W)), self._n(m + ".conv"): TensorSpec((rows, self.taps), role="filter")})
+        specs.update({self._n("b"): TensorSpec((N, W)), self._n("A_log"): TensorSpec((N,), role="bias"),
+                      self._n("norm"): TensorSpec((self.v_head_dim,), role="norm"), self._n("a"): TensorSpec((N, W)),
+                      self._n("dt_bias"): TensorSpec((N,), role="bias"), self._n("g"): TensorSpec((NV, W)), self._n("o"): TensorSpec((W, NV))})
+        return specs
+
+    def bind(self, tensors):
+        # everything that reads h is one product: q, k, v, the gate, the write strengths and the decays (and rows of zeros at the end)
+        rows = torch.cat([tensors[self._n(m)] for m in ("q", "k", "v", "g", "b", "a")], dim=0)
+        pad = -rows.shape[0] % self.ROW_MULTIPLE
+        self.proj = Linear(self._matrix(torch.cat([rows, rows.new_zeros(pad, rows.shape[1])], dim=0)), None, self.rt)
+        self.conv = self._vector_f32(torch.cat([tensors[self._n(m + ".conv")] for m in "qkv"], dim=0))
+        self.decay_rate = self._vector_f32(torch.exp(tensors[self._n("A_log")].to(torch.float64)))
+        self.dt = self._vector_f32(tensors[self._n("dt_bias")])
+        self.norm = self._vector_f32(tensors[self._n("norm")])
+        self.o = Linear(self._matrix(tensors[self._n("o")]), None, self.rt)
+
+    def cache_spec(self):
+        n = self.num_heads * self.head_dim * self.v_head_dim + self.taps * self._conv_channels()
+        return StateSpec((n + -n % 4,), torch.float32)              # the heads' matrices, then the ring of the convolutions' last inputs
+
+    def in_width(self):
+        n = self._conv_channels() + self.num_heads * (self.v_head_dim + 2)
+        return n + -n % self.ROW_MULTIPLE
+
+    def out_width(self):
+        return self.num_heads * self.v_head_dim
+
+    def mix(self, p, col, batch, cache, out=None):
+        """p fp32 [T, >= col + in_width]: [q | k | v | g | b | a] from column ``col``; returns the gated heads [T, N*V] (or writes them into
+        ``out`` = (matrix, first column))."""
+        N, M, K, V = self.num_heads, self.num_qk_heads, self.head_dim, self.v_head_dim
+        g_col = col + self._conv_channels()
+        b_col, a_col = g_col + N * V, g_col + N * V + N
+        if kernels.token_state_supports(batch, K, V, True):            # a step of single tokens: one kernel
+            return kernels.gated_delta_token(p, col, g_col, b_col, a_col, self.conv, self.decay_rate, self.dt, batch, cache.state, N, M, K, V,
+                                             self.norm, self.eps, self.rt.dtype, out=out)
+        qkv, g, beta = kernels.gated_delta_prepare(p, col, b_col, a_col, self.conv, self.decay_rate, self.dt, batch, cache.state, N, M, K, V)
+        o = kernels.gated_delta_scan(qkv, g, beta, batch, cache.state, N, M, K, V)
+        return kernels.head_finish(o, self.norm, (p, g_col), N, V, self.eps, "silu", self.rt.dtype, out=out)
+
+    def forward(self, x, batch, cache, residual):
+        """Adds the mixer's output into ``residual``, or (``residual`` None) returns it as a new fp32 [T, W]."""
+        return self.o.forward(self.mix(self.proj.forward(x), 0, batch, cache), accumulate_into=residual)
+
+
+class LightningMixer(Part):
+    graph_safe = True       # request boundaries and state rows come from the batch's device tensors (q_start, slots)
+
+    def __init__(self, rt, hidden_size, num_heads, head_dim, decay, eps, v_head_dim=None, prefix="mix."):
+        """``decay``: one number per head."""
+        if head_dim > 256:
+            raise ConfigError(f"the lightning mixer takes heads of up to 256 key channels, not {head_dim}")
+        if len(decay) != num_heads:
+            raise ConfigError(f"lightning attention: {len(decay)} decays for {num_heads} heads")
+        self.rt, self.hidden_size, self.num_heads, self.head_dim = rt, hidden_size, num_heads, head_dim
+        self.v_head_dim = head_dim if v_head_dim is None else v_head_dim
+        self.eps, self.prefix = float(eps), prefix
+        self.decay = torch.tensor([float(g) for g in decay], dtype=torch.float64).to(torch.float32).to(rt.device)
+
+    def _n(self, short):
+        return self.prefix + short
+
+    def tensor_specs(self):
+        W, NK, NV = self.hidden_size, self.num_heads * self.head_dim, self.num_heads * self.v_head_dim
+        return {self._n("q"): TensorSpec((NK, W)), self._n("k"): TensorSpec((NK, W)), self._n("v"): TensorSpec((NV, W)),
+                self._n("g"): TensorSpec((NV, W)), self._n("o"): TensorSpec((W, NV)), self._n("norm"): TensorSpec((NV,), role="norm")}
+
+    def bind(self, tensors):
+        # q, k, v and the gate read the same input: one product
+        self.proj = Linear(self._matrix(torch.cat([tensors[self._n(m)] for m in ("q", "k", "v", "g")], dim=0)), None, self.rt)
+        self.norm = self._vector_f32(tensors[self._n("norm")])
+        self.o = Linear(self._matrix(tensors[self._n("o")]), None, self.rt)
+
+    def cache_spec(self):
+        n = self.num_heads * self.head_dim * self.v_head_dim
+        return StateSpec((n + -n % 4,), torch.float32)
+
+    def in_width(self):
+        return 2 * self.num_heads * (self.head_dim + self.v_head_dim)
+
+    def out_width(self):
+        return self.num_heads * self.v_head_dim
+
+    def mix(self, p, col, batch, cache, out=None):
+        """p fp32 [T, >= col + in_width]: [q | k | v | g] from column ``col`` (portions: q, k, v are overwritten); returns the normed and
+        gated heads [T, N*V] (or writes them into ``out`` = (matrix, first column))."""
+        N, K, V = self.num_heads, self.head_dim, self.v_head_dim
+        scan = kernels.lightning_token if kernels.token_state_supports(batch, K, V, False) else kernels.lightning_scan
+        o = scan(p, col, self.decay, batch, cache.state, N, K, V)
+        return kernels.gated_rows(o, self.norm, (p, col + N * (2 * K + V)), self.eps, self.rt.dtype, out=out)
+
+    def forward(self, x, batch, cache, residual):
+        """Adds the mixer's output into ``residual``, or (``residual`` None) returns it as a new fp32 [T, W]."""
+        return self.o.forward(self.mix(self.proj.forward(x), 0, batch, cache), accumulate_into=residual)
+
+
+register_part("mixer", "gated_delta", GatedDeltaMixer, replace=True)
+register_part("mixer", "lightning", LightningMixer, replace=True)
 register_part("mixer", "gated_linear", GatedLinearMixer, replace=True)
 register_part("mixer", "retention", RetentionMixer, replace=True)
 register_part("mixer", "gated_write", GatedWriteMixer, replace=True)

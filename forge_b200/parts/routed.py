@@ -4,7 +4,8 @@
     y = sum over the chosen e of s_e * Wdown_e (silu(Wgate_e x) * (Wup_e x))          (s_e divided by their sum with ``renormalize``)
 
 Options: experts may be ranked by s + ``correction`` (a number per expert; the weights stay s); the experts may be cut into ``groups``
-consecutive blocks of equal size, each ranked by the largest ranking number in it, of which only the ``keep`` best take part; the weights
+consecutive blocks of equal size, each ranked by the largest ranking number in it (or by the sum of its ``group_top`` = 2 largest), of
+which only the ``keep`` best take part; the weights
 may be multiplied by ``route_scale``; a ``shared`` feed-forward (any feed-forward part) may run for every token and be added.
 
 The router's arithmetic is fp32.  Three paths, all with everything but the last one's row counts read from device memory:
@@ -29,11 +30,12 @@ from .linear import Linear
 
 class RoutedExperts(Part):
     graph_safe = True
+    adds_in_product = False    # the experts' weighted sum is a kernel of its own: its result joins the stream in another
     SORTED_FROM = 128          # tokens in a step from which the pairs are ranked by expert
     BY_EXPERT_FROM = 2         # ... and from which the path by pairs goes expert by expert (the same numbers, fewer reads)
 
     def __init__(self, rt, hidden_size, intermediate_size, experts, top, score="sigmoid", renormalize=False, prefix="mlp.",
-                 correction=False, groups=0, keep=0, route_scale=1.0, shared=None):
+                 correction=False, groups=0, keep=0, route_scale=1.0, shared=None, group_top=1):
         """``shared``: the PartSpec of a feed-forward part that every token passes through beside its experts, or None."""
         if not 1 <= top <= experts:
             raise ConfigError(f"routed feed-forward: {top} of {experts} experts")
@@ -41,6 +43,9 @@ class RoutedExperts(Part):
         if groups > 1 and (experts % groups or not 1 <= keep <= groups or top > keep * (experts // groups)):
             raise ConfigError(f"routed feed-forward: {experts} experts in {groups} groups of which {keep} are kept cannot give {top} a token")
         self.correction, self.groups, self.keep, self.route_scale = bool(correction), groups if groups > 1 else 0, keep, float(route_scale)
+        if group_top not in (1, 2):
+            raise ConfigError(f"routed feed-forward: a block of experts is ranked by its largest or its two largest numbers, not {group_top}")
+        self.group_top = int(group_top)
         self.shared = None if shared is None else build_part("feed_forward", shared, rt)
         self.bias = None
         if score not in ("sigmoid", "softmax"):
@@ -116,7 +121,7 @@ class RoutedExperts(Part):
     def forward(self, x, residual):
         """Adds the output into ``residual`` fp32 [T, W], or (``residual`` None) returns it as a new fp32 [T, W]."""
         idx, wts = kernels.moe_route(x, self.router, self.top, softmax=self.score == "softmax", renorm=self.renormalize,
-                                     correction=self.bias, groups=self.groups, keep=self.keep, factor=self.route_scale)
+                                     correction=self.bias, groups=self.groups, keep=self.keep, factor=self.route_scale, group_top=self.group_top)
         T = x.shape[0]
         tensor_core = self.gate_up_of[0].tensor_core and self.down_of[0].tensor_core
         if T >= self.SORTED_FROM and not torch.cuda.is_current_stream_capturing():

@@ -11,8 +11,11 @@ Rotary positions on the first ``rotary_dims`` channels of every map, channel i p
 key channels) with a weight per channel; a query temperature 1 + coef ln(floor((p + 1) / every) + 1) at position p; and
     score(i, j) = scale q(i) . k(j) - r1_h ln(1 + r2_h (i - j))
 
-"masked_attention": no rotation (positions do not enter the scores); optional biases in q, k and v; the scale is a parameter;
-optionally  score <- softcap tanh(score / softcap);  and a position i sees j <= i only
+"masked_attention": optional biases in q, k and v; optionally a rotation of q and k (a position part with ``inv_freq`` that pairs
+channel i with i + half, its ``amplitude`` on cos and sin; without one positions do not enter the scores) and then (``qk_norm``) every
+query and key head divided by its root mean square; the scale is a parameter; optionally  score <- softcap tanh(score / softcap);
+optionally a ``sink`` (one learned number per head, b_h: the softmax denominator becomes sum_j exp(score_j) + exp(b_h)); and a position i
+sees j <= i only
     within a sliding ``window``  (i - window < j),  or  within its own ``chunk``  (i // chunk == j // chunk),
 chunks counted from the sequence's first position.  Pages whose keys no future query sees go back to the pool.
 
@@ -155,15 +158,25 @@ class DistanceBiasAttention(_ScoredAttention):
 
 class MaskedAttention(_ScoredAttention):
     def __init__(self, rt, hidden_size, num_heads, num_kv_heads, head_dim, v_head_dim=None, scale=None, window=None, chunk=None,
-                 softcap=None, qkv_bias=False, out_scale=1.0, prefix="mix."):
+                 softcap=None, qkv_bias=False, out_scale=1.0, prefix="mix.", position=None, qk_norm=False, eps=0.0, sink=False):
         """``window`` / ``chunk``: None or a number of positions (both may be given: a key must pass both); ``softcap``: None or the
-        cap; ``qkv_bias``: tensors ``q.b``, ``k.b``, ``v.b`` are added in the projection."""
+        cap; ``qkv_bias``: tensors ``q.b``, ``k.b``, ``v.b`` are added in the projection; ``position``: the PartSpec of the rotation or
+        None; ``qk_norm``: q and k heads are divided by their root mean square (``eps`` inside the root); ``sink``: a tensor ``sink``."""
         self._sizes(rt, hidden_size, num_heads, num_kv_heads, head_dim, v_head_dim, scale, out_scale, prefix)
         self.window, self.chunk = (int(window) if window else None), (int(chunk) if chunk else None)
         self.softcap, self.qkv_bias = (float(softcap) if softcap else None), bool(qkv_bias)
         if (self.window is not None and self.window < 1) or (self.chunk is not None and self.chunk < 1) or \
                 (self.softcap is not None and not self.softcap > 0.0):
             raise ConfigError(f"masked attention: window {window}, chunk {chunk}, softcap {softcap}")
+        self.position = None if position is None else build_part("position", position, rt)
+        if self.position is not None and not (hasattr(self.position, "inv_freq") and self.position.halves):
+            raise ConfigError("this attention rotates inside its own prepare step and needs a position part with 'inv_freq' that pairs "
+                              "channels half the rotated ones apart")
+        self.qk_norm, self.eps, self.sink = bool(qk_norm), float(eps), bool(sink)
+        self.sinks = None
+
+    def sub_parts(self):
+        return [] if self.position is None else [self.position]
 
     def tensor_specs(self):
         W, H, G, D, E = self.hidden_size, self.num_heads, self.num_kv_heads, self.head_dim, self.v_head_dim
@@ -172,10 +185,13 @@ class MaskedAttention(_ScoredAttention):
         if self.qkv_bias:
             specs.update({self._n("q.b"): TensorSpec((H * D,), role="bias"), self._n("k.b"): TensorSpec((G * D,), role="bias"),
                           self._n("v.b"): TensorSpec((G * E,), role="bias")})
+        if self.sink:
+            specs[self._n("sink")] = TensorSpec((H,), role="bias")
         return specs
 
     def bind(self, tensors):
         rows = torch.cat([tensors[self._n(m)] for m in "qkv"], dim=0)
+        self.sinks = self._vector_f32(tensors[self._n("sink")]) if self.sink else None
         b = self._vector_f32(torch.cat([tensors[self._n(m + ".b")].float() for m in "qkv"])) if self.qkv_bias else None
         self.proj = Linear(self._matrix(rows), b, self.rt)              # q, k, v in one product, the biases in its epilogue
         self.o = Linear(self._matrix(tensors[self._n("o")]), None, self.rt)
@@ -193,10 +209,15 @@ class MaskedAttention(_ScoredAttention):
         [T, H*E] (or writes them into ``out`` = (matrix, first column))."""
         H, G, D, E = self.num_heads, self.num_kv_heads, self.head_dim, self.v_head_dim
         g = batch.groups[cache.group]
-        q = kernels.scored_prepare(proj, batch.positions, g.slot_mapping if cache.writable else None,
-                                   cache.kv if cache.writable else None, H, G, 1, D, E, cache.page_size, self.rt.dtype, col=col)
+        where = (batch.positions, g.slot_mapping if cache.writable else None, cache.kv if cache.writable else None)
+        if self.position is None and not self.qk_norm:
+            q = kernels.scored_prepare(proj, *where, H, G, 1, D, E, cache.page_size, self.rt.dtype, col=col)
+        else:
+            freq, amp = (None, 1.0) if self.position is None or not self.position.rotary_dims else (self.position.inv_freq, self.position.amplitude)
+            q = kernels.scored_prepare_heads(proj, *where, H, G, D, E, cache.page_size, self.rt.dtype, inv_freq=freq, amp=amp, norm=self.qk_norm,
+                                             eps=self.eps, col=col)
         return kernels.scored_attention(q, cache.kv, g, batch, H, G, 1, D, E, cache.page_size, self.scale, out_scale=self.out_scale,
-                                        out=out, window=self.window or 0, chunk=self.chunk or 0, softcap=self.softcap or 0.0)
+                                        out=out, window=self.window or 0, chunk=self.chunk or 0, softcap=self.softcap or 0.0, sink=self.sinks)
 
 
 register_part("mixer", "differential_attention", DifferentialAttention, replace=True)

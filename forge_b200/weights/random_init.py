@@ -44,6 +44,10 @@ def random_tensors(config, seed=0, std=0.02, embed_std=None, norm_std=0.0, bias_
             out[name] = t.to(dtype)
         elif spec.role == "route_bias":       # what is added to a router's scores (of order 1 / experts) before the choice
             out[name] = (0.05 * torch.randn(spec.shape, generator=gen, dtype=torch.float32, device=device)).to(dtype)
+        elif spec.role == "filter":           # a short convolution over time: mostly the current token, some of the ones before
+            t = 0.3 * torch.randn(spec.shape, generator=gen, dtype=torch.float32, device=device)
+            t[:, -1] += 1.0
+            out[name] = t.to(dtype)
         elif spec.role == "lambda_part":      # vectors whose pairwise dot products are exponentiated: keep those of order 1/2
             n = max(1, int(torch.tensor(spec.shape).prod()))
             out[name] = (torch.randn(spec.shape, generator=gen, dtype=torch.float32, device=device) * (0.7 / n ** 0.25)).to(dtype)
