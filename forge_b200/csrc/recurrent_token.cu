@@ -24,6 +24,10 @@ __device__ __forceinline__ float sigmoidf(float x) { return 1.0f / (1.0f + expf(
 __device__ __forceinline__ float siluf(float x) { return x * sigmoidf(x); }
 __device__ __forceinline__ float softplusf(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
+// exp(-x) of a small x is a number just below one that hundreds of tokens multiply: 1 + (exp(-x) - 1) is it to the last bit, where an
+// error of one unit there would be the same for every token and add up.
+__device__ __forceinline__ float decayf(float x) { return 1.0f + expm1f(-x); }
+
 struct ShortConv {
     const float* w;                   // fp32 [channels, taps], the last column is the current token's; null: no convolution
     int taps;
@@ -92,7 +96,7 @@ delta_prepare_kernel(const DeltaPrepare d) {
     if (lane == 0) {
         const float* row = d.p.p + (size_t)t * d.p.ld;
         d.beta[(size_t)t * d.N + head] = sigmoidf(row[d.b_col + head]);
-        d.g[(size_t)t * d.N + head] = expf(-d.decay_rate[head] * softplusf(row[d.a_col + head] + d.dt[head]));
+        d.g[(size_t)t * d.N + head] = decayf(d.decay_rate[head] * softplusf(row[d.a_col + head] + d.dt[head]));
     }
 }
 
@@ -245,7 +249,7 @@ token_state_kernel(const TokenState d, TA* __restrict__ out, long long out_ld) {
             vs[i] = siluf(convolve(d.cv, d.v.p + c, d.v.ld, t, t, pos, cc, ring));
             now[cc] = d.v.p[(size_t)t * d.v.ld + c];
         }
-        g = expf(-d.decay[head] * softplusf(d.a.p[(size_t)t * d.a.ld + head] + d.dt[head]));
+        g = decayf(d.decay[head] * softplusf(d.a.p[(size_t)t * d.a.ld + head] + d.dt[head]));
         beta = sigmoidf(d.b.p[(size_t)t * d.b.ld + head]);
         qq = forge::warp_sum(qq);
         kk = forge::warp_sum(kk);
