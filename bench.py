@@ -162,7 +162,7 @@ def main():
     ap.add_argument("--no-points", action="store_true", help="skip batch 1 / 64 and the prefill")
     ap.add_argument("--no-shapes", action="store_true", help="skip the Llama-3-8B and Qwen2.5-7B shaped points")
     ap.add_argument("--block-size", type=int, default=64, help="tokens per cache page (named in config)")
-    ap.add_argument("--design", default=None, choices=["zatupel", "tidenex", "tuzavik", "natalorn", "ramupel"],
+    ap.add_argument("--design", default=None, choices=["zatupel", "tidenex", "tuzavik", "natalorn", "ramupel", "zuretar"],
                     help="instead of the default workload: prefill and decode speed of that design at a few layer sizes, "
                          "beside the LLaMA decoder of equal width, depth and head counts")
     a = ap.parse_args()
@@ -758,8 +758,83 @@ class RamupelBench(ShapeBench):
         return flops
 
 
+def zuretar_shape(width, layers, heads, kv_heads, dim, ff, state_heads, state_dim, window, vocab, **_):
+    """A Zuretar configuration at a real model's layer sizes, in turn: a delta layer (``state_heads`` heads of ``state_dim``, two of which share
+    a query/key head, convolutions over four tokens) with a dense feed-forward, one with routed experts, a parallel layer (attention in
+    chunks of ``window`` beside lightning attention) with routed experts, and the first layer's weights again; 8 experts of half the
+    dense width in 4 groups of which 2 are kept, 2 a token, so that a token passes through as many feed-forward weights as in the
+    dense layers."""
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": ff // 2}, "router": {"experts": 8, "top": 2, "groups": {"count": 4, "keep": 2}}}
+    delta = {"type": "delta", "mixer": {"heads": state_heads, "kv_heads": state_heads // 2, "dim": state_dim, "vdim": state_dim, "conv": 4}}
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "mask": {"size": window}, "scale": dim ** -0.5,
+            "rot": {"dims": dim, "base": 10000.0, "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}}
+    right = {"heads": state_heads, "dim": state_dim, "vdim": state_dim, "decay": [1.0 - 2.0 ** (-3.0 - 5.0 * i / state_heads) for i in range(state_heads)]}
+    pair = {"type": "parallel", "mixer": {"left": left, "right": right}}
+    turn = [dict(delta, mlp=dense), dict(delta, mlp=moe), dict(pair, mlp=moe)]
+    return {"architecture": "Zuretar", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "max_positions": 8192,
+            "layers": [dict(turn[0], weights_of=i - 3) if i % 4 == 3 else turn[i % 4] for i in range(layers)]}
+
+
+def zuretar_matmul_params(cfg, experts_read=None):
+    """Matrix elements of all layers as they run that a token passes through (``experts_read`` None: its ``top`` experts) or that a step
+    reads (``experts_read``: how many experts of a routed layer), and of the head."""
+    W, total = cfg.width, 0
+    for layer in cfg.layers:
+        m = layer["mixer"]
+        if layer["type"] == "delta":
+            N, QK, NV = m["heads"], m["kv_heads"] * m["dim"], m["heads"] * m["vdim"]
+            total += W * (2 * QK + 2 * NV + 2 * N) + W * NV + m["conv"] * (2 * QK + NV)
+        else:
+            a, b = m["left"], m["right"]
+            total += W * (a["heads"] * a["dim"] + a["kv_heads"] * (a["dim"] + a["vdim"])) + W * a["heads"] * a["vdim"]
+            total += W * b["heads"] * 2 * (b["dim"] + b["vdim"]) + W * b["heads"] * b["vdim"]
+        mlp = layer.get("mlp")
+        if mlp and mlp["kind"] == "dense":
+            total += 3 * W * mlp["ff"]
+        elif mlp:
+            n = mlp["router"]["top"] if experts_read is None else min(mlp["router"]["experts"], experts_read)
+            total += 3 * W * mlp["expert"]["ff"] * n + W * mlp["router"]["experts"]
+    return total, cfg.vocab * W
+
+
+class ZuretarBench(ShapeBench):
+    """ShapeBench's measurements for a Zuretar configuration: only bytes and FLOPs are counted otherwise."""
+
+    def decode_bytes(self, B, ctx):
+        """Every matrix once per run of its layer (of a routed layer the experts that B tokens can choose), and per request the keys and
+        values of the position's chunk and the state matrices and the convolutions' inputs, read and written."""
+        cfg = self.cfg
+        top = max([l["mlp"]["router"]["top"] for l in cfg.layers if l.get("mlp") and l["mlp"]["kind"] == "moe"] or [1])
+        layers, head = zuretar_matmul_params(cfg, experts_read=B * top)
+        total = 2 * (layers + head)
+        for layer in cfg.layers:
+            m = layer["mixer"]
+            if layer["type"] == "delta":
+                total += B * 4 * (2 * m["heads"] * m["dim"] * m["vdim"] + m["conv"] * (2 * m["kv_heads"] * m["dim"] + m["heads"] * m["vdim"]))
+            else:
+                a, b = m["left"], m["right"]
+                total += B * (ctx % a["mask"]["size"] + 1) * a["kv_heads"] * (a["dim"] + a["vdim"]) * 2 + B * 2 * 4 * b["heads"] * b["dim"] * b["vdim"]
+        return total
+
+    def prefill_flops(self, T):
+        """Products, the attention as the design states it (per visible pair and head: scores over dim channels, values of vdim), and the
+        recurrences token by token: 6 FLOPs per state element of the delta rule, 4 of lightning attention."""
+        cfg = self.cfg
+        layers, head = zuretar_matmul_params(cfg)
+        flops = 2 * T * layers + 2 * head
+        for layer in cfg.layers:
+            m = layer["mixer"]
+            if layer["type"] == "delta":
+                flops += 6 * T * m["heads"] * m["dim"] * m["vdim"]
+            else:
+                a, b = m["left"], m["right"]
+                flops += 2 * _visible_pairs(T, chunk=a["mask"]["size"]) * a["heads"] * (a["dim"] + a["vdim"]) + 4 * T * b["heads"] * b["dim"] * b["vdim"]
+        return flops
+
+
 def design_arm(a):
-    """Prefill and decode speed of the Zatupel, Tidenex, Tuzavik, Natalorn or Ramupel design at a few layer sizes (random weights), each beside the LLaMA decoder
+    """Prefill and decode speed of the Zatupel, Tidenex, Tuzavik, Natalorn, Ramupel or Zuretar design at a few layer sizes (random weights), each beside the LLaMA decoder
     of the same width, depth, head counts and feed-forward width run the same way: decode device-timed at batch 1, 8 and
     64 after 512-token prompts, one prompt step of 2,048 tokens.  One JSON line."""
     import torch
@@ -793,6 +868,9 @@ def design_arm(a):
             arms = [("natalorn", natalorn_shape(**z), NatalornBench), ("tuzavik", tuzavik_shape(**z), TuzavikBench), arms[1]]
         if a.design == "ramupel":         # beside the design whose latent attention and state scan are the nearest, and the plain decoder
             arms = [("ramupel", ramupel_shape(**z), RamupelBench), ("tuzavik", tuzavik_shape(**z), TuzavikBench), arms[1]]
+        if a.design == "zuretar":         # beside the designs whose parallel layers, and whose chunked attention and experts, are the nearest
+            arms = [("zuretar", zuretar_shape(**z), ZuretarBench), ("ramupel", ramupel_shape(**z), RamupelBench),
+                    ("natalorn", natalorn_shape(**z), NatalornBench), arms[1]]
         for arch, shape, maker in arms:
             b = maker(shape, PROMPT_LEN, 64, steps, a.warmup, a.block_size, prefill_tokens=PREFILL_TOKENS)
             r = {}

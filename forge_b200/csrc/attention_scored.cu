@@ -92,71 +92,81 @@ scored_prepare_kernel(const float* __restrict__ proj, int ld, const int32_t* __r
 
 constexpr int kHeadRegs = 8;           // rotated pairs, and twice as many channels that pass, that a lane holds of a head at most
 
-// One warp per (token, head): the QU query heads, the KU key heads (both D channels) and the KU value heads (E channels) of fp32 row
-// [q | k | v].  A query or key head's first rot_dims channels turn by position * inv_freq (channel i with i + rot_dims/2; cos and sin
-// times amp), then (norm) the head is divided by its root mean square.  Queries go to q_out, keys and values to their cache rows.
+// A warp per head: the QU query heads, the KU key heads (both D channels) and the KU value heads (E channels) of fp32 row [q | k | v].  A
+// query or key head's first rot_dims channels turn by position * inv_freq (channel i with i + rot_dims/2; cos and sin times amp), then
+// (norm) the head is divided by its root mean square.  Queries go to q_out, keys and values to their cache rows.  A CTA takes one token
+// (steps of few tokens: a share of its heads); the token's sines and cosines are worked out once for all of them.
 template <typename TC>
 __global__ void __launch_bounds__(kPrepThreads)
 scored_prepare_heads_kernel(const float* __restrict__ proj, int ld, const int32_t* __restrict__ positions,
                             const int32_t* __restrict__ slot_mapping, const float* __restrict__ inv_freq, float amp, TC* __restrict__ q_out,
                             TC* __restrict__ cache, int QU, int KU, int D, int E, int rot_dims, int norm, float eps, int page_size,
                             long long page_stride) {
+    __shared__ float sn[32 * kHeadRegs], cs[32 * kHeadRegs];
     forge::pdl_launch_dependents();
     forge::pdl_wait();
-    const int t = blockIdx.x, lane = threadIdx.x & 31, unit = blockIdx.y * (kPrepThreads / 32) + (threadIdx.x >> 5);
-    if (unit >= QU + 2 * KU) return;
+    const int t = blockIdx.x, lane = threadIdx.x & 31, half = rot_dims >> 1;
     const int slot = slot_mapping ? slot_mapping[t] : -1;
     const bool store = slot >= 0 && FORGE_SLOT_OK(slot);
     const int page = store ? slot / page_size : 0, off = store ? slot % page_size : 0;
     TC* kbase = cache + (size_t)page * page_stride;
-    if (unit >= QU + KU) {                     // a value head passes as it is
-        if (!store) return;
-        const int g = unit - QU - KU;
-        const float* v = proj + (size_t)t * ld + (size_t)(QU + KU) * D + (size_t)g * E;
-        TC* dst = kbase + (size_t)KU * page_size * D + ((size_t)g * page_size + off) * E;
-        for (int c = lane; c < E; c += 32) dst[c] = forge::from_float<TC>(v[c]);
-        return;
-    }
-    if (unit >= QU && !store) return;
-    const float* x = proj + (size_t)t * ld + (size_t)unit * D;
-    TC* dst = unit < QU ? q_out + ((size_t)t * QU + unit) * D : kbase + ((size_t)(unit - QU) * page_size + off) * D;
-    const int half = rot_dims >> 1;
     const float pos = (float)positions[t];
-    float lo[kHeadRegs], hi[kHeadRegs], pass[2 * kHeadRegs], ss = 0.f;
-#pragma unroll
-    for (int i = 0; i < kHeadRegs; ++i) {
-        const int c = lane + 32 * i;
-        lo[i] = hi[i] = 0.f;
-        if (c < half) {
-            float s, cs;
-            sincosf(pos * inv_freq[c], &s, &cs);
-            s *= amp;
-            cs *= amp;
-            const float u = x[c], v = x[c + half];
-            lo[i] = u * cs - v * s;
-            hi[i] = v * cs + u * s;
-            ss = fmaf(lo[i], lo[i], fmaf(hi[i], hi[i], ss));
+    for (int i = threadIdx.x; i < half; i += kPrepThreads) {
+        float s, c;
+        sincosf(pos * inv_freq[i], &s, &c);
+        sn[i] = s * amp;
+        cs[i] = c * amp;
+    }
+    __syncthreads();
+    const int warps = kPrepThreads / 32;
+    for (int unit = blockIdx.y * warps + (threadIdx.x >> 5); unit < QU + 2 * KU; unit += gridDim.y * warps) {
+        if (unit >= QU + KU) {                     // a value head passes as it is
+            if (!store) continue;
+            const int g = unit - QU - KU;
+            const float* v = proj + (size_t)t * ld + (size_t)(QU + KU) * D + (size_t)g * E;
+            TC* dst = kbase + (size_t)KU * page_size * D + ((size_t)g * page_size + off) * E;
+            for (int c = lane; c < E; c += 32) dst[c] = forge::from_float<TC>(v[c]);
+            continue;
         }
-    }
+        if (unit >= QU && !store) continue;
+        const float* x = proj + (size_t)t * ld + (size_t)unit * D;
+        TC* dst = unit < QU ? q_out + ((size_t)t * QU + unit) * D : kbase + ((size_t)(unit - QU) * page_size + off) * D;
+        float lo[kHeadRegs], hi[kHeadRegs], pass[2 * kHeadRegs], ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < 2 * kHeadRegs; ++i) {
-        const int c = rot_dims + lane + 32 * i;
-        pass[i] = c < D ? x[c] : 0.f;
-        ss = fmaf(pass[i], pass[i], ss);
-    }
-    const float inv = norm ? 1.0f / sqrtf(forge::warp_sum(ss) / (float)D + eps) : 1.0f;
-#pragma unroll
-    for (int i = 0; i < kHeadRegs; ++i) {
-        const int c = lane + 32 * i;
-        if (c < half) {
-            dst[c] = forge::from_float<TC>(lo[i] * inv);
-            dst[c + half] = forge::from_float<TC>(hi[i] * inv);
+        for (int i = 0; i < kHeadRegs; ++i) {
+            if (32 * i >= half) break;             // (the same for the whole warp)
+            const int c = lane + 32 * i;
+            lo[i] = hi[i] = 0.f;
+            if (c < half) {
+                const float u = x[c], v = x[c + half];
+                lo[i] = u * cs[c] - v * sn[c];
+                hi[i] = v * cs[c] + u * sn[c];
+                ss = fmaf(lo[i], lo[i], fmaf(hi[i], hi[i], ss));
+            }
         }
-    }
 #pragma unroll
-    for (int i = 0; i < 2 * kHeadRegs; ++i) {
-        const int c = rot_dims + lane + 32 * i;
-        if (c < D) dst[c] = forge::from_float<TC>(pass[i] * inv);
+        for (int i = 0; i < 2 * kHeadRegs; ++i) {
+            if (rot_dims + 32 * i >= D) break;
+            const int c = rot_dims + lane + 32 * i;
+            pass[i] = c < D ? x[c] : 0.f;
+            ss = fmaf(pass[i], pass[i], ss);
+        }
+        const float inv = norm ? 1.0f / sqrtf(forge::warp_sum(ss) / (float)D + eps) : 1.0f;
+#pragma unroll
+        for (int i = 0; i < kHeadRegs; ++i) {
+            if (32 * i >= half) break;
+            const int c = lane + 32 * i;
+            if (c < half) {
+                dst[c] = forge::from_float<TC>(lo[i] * inv);
+                dst[c + half] = forge::from_float<TC>(hi[i] * inv);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < 2 * kHeadRegs; ++i) {
+            if (rot_dims + 32 * i >= D) break;
+            const int c = rot_dims + lane + 32 * i;
+            if (c < D) dst[c] = forge::from_float<TC>(pass[i] * inv);
+        }
     }
 }
 
@@ -366,7 +376,7 @@ extern "C" int forge_scored_prepare_heads(const float* proj, int ld, const int32
     const int units = QU + 2 * KU, warps = kPrepThreads / 32;
     cudaError_t e = cudaSuccess;
     FORGE_DISPATCH_DTYPE(dtype, TT,
-        e = forge::launch(scored_prepare_heads_kernel<TT>, dim3(T, (units + warps - 1) / warps), dim3(kPrepThreads), 0, stream, 1, proj, ld,
+        e = forge::launch(scored_prepare_heads_kernel<TT>, dim3(T, T >= 256 ? 1 : (units + warps - 1) / warps), dim3(kPrepThreads), 0, stream, 1, proj, ld,
                           positions, slot_mapping, inv_freq, amp, (TT*)q_out, (TT*)cache, QU, KU, D, E, rot_dims, norm, eps, page_size,
                           page_stride));
     return forge::check_launch("scored_prepare_heads", e);

@@ -43,11 +43,11 @@ template <> __device__ __forceinline__ void store_pack<__nv_bfloat16, 4>(__nv_bf
     *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
 }
 
-// One CTA per row; thread i takes the packs i, i + blockDim, ... of V channels in every walk, so what it keeps of x in shared memory
-// (W floats) it reads back itself.  The normed terms are read twice, the second time from the cache.
+// One CTA per row; thread i takes the packs i, i + blockDim, ... of V channels in every walk, so what it keeps in shared memory (the
+// normed terms, W floats each, if they fit: `keep`; and the new x) it reads back itself.
 template <typename TOut, int V>
 __global__ void __launch_bounds__(kMaxThreads)
-join_kernel(const Join d, TOut* __restrict__ h) {
+join_kernel(const Join d, TOut* __restrict__ h, int keep) {
     using P = typename Pack<V>::type;
     extern __shared__ __align__(16) float u[];
     __shared__ float red[32];
@@ -58,11 +58,14 @@ join_kernel(const Join d, TOut* __restrict__ h) {
     float factor[kMaxTerms], part[kMaxTerms];
 #pragma unroll
     for (int k = 0; k < kMaxTerms; ++k) part[k] = 0.f;
+    float* kept = u + W;               // [term][W]
+#pragma unroll 2
     for (int i = threadIdx.x; i < packs; i += blockDim.x) {
 #pragma unroll
         for (int k = 0; k < kMaxTerms; ++k) {
             if (k >= d.n || !d.term[k].w) continue;
             P y = __ldg(reinterpret_cast<const P*>(d.term[k].y + row) + i);
+            if (keep) *reinterpret_cast<P*>(kept + (size_t)k * W + (size_t)i * V) = y;
 #pragma unroll
             for (int e = 0; e < V; ++e) part[k] = fmaf(lane_of(y, e), lane_of(y, e), part[k]);
         }
@@ -80,7 +83,8 @@ join_kernel(const Join d, TOut* __restrict__ h) {
 #pragma unroll
         for (int k = 0; k < kMaxTerms; ++k) {
             if (k >= d.n) continue;
-            P y = __ldg(reinterpret_cast<const P*>(d.term[k].y + row) + i);
+            P y = keep && d.term[k].w ? *reinterpret_cast<const P*>(kept + (size_t)k * W + (size_t)i * V)
+                                      : __ldg(reinterpret_cast<const P*>(d.term[k].y + row) + i);
             if (d.term[k].w) {
                 P w = __ldg(reinterpret_cast<const P*>(d.term[k].w) + i);
 #pragma unroll
@@ -118,11 +122,17 @@ cudaError_t run(const Join& d, void* h, int T, cudaStream_t stream) {
         if (e != cudaSuccess) return e;
         done = true;
     }
-    // few rows: as many threads as the row has packs, so that a walk is one trip to memory; many rows: 128
+    // few rows: as many threads as the row has packs, so that a walk is one trip to memory; many rows: two packs a thread
     int threads = (d.W / V + 31) / 32 * 32;
-    const int most = T <= 148 ? kMaxThreads : 128;
-    threads = threads < 32 ? 32 : (threads > most ? most : threads);
-    return forge::launch(join_kernel<TOut, V>, dim3(T), dim3(threads), d.next_w ? sizeof(float) * (size_t)d.W : 0, stream, 1, d, (TOut*)h);
+    if (T > 148) threads = (threads / 2 + 31) / 32 * 32;
+    threads = threads < 32 ? 32 : (threads > kMaxThreads ? kMaxThreads : threads);
+    int last = 0;                       // terms up to the last normed one have room in shared memory
+    for (int k = 0; k < d.n; ++k)
+        if (d.term[k].w) last = k + 1;
+    size_t smem = sizeof(float) * (size_t)d.W * (1 + last);
+    const int keep = last > 0 && smem <= 64 * 1024 ? 1 : 0;
+    if (!keep) smem = sizeof(float) * (size_t)d.W;
+    return forge::launch(join_kernel<TOut, V>, dim3(T), dim3(threads), d.next_w || keep ? smem : 0, stream, 1, d, (TOut*)h, keep);
 }
 
 }  // namespace

@@ -16,12 +16,9 @@
 //   gated linear attention:    S <- diag(a_t) S + k_t v_t^T ;   o_t = K^-1/2 S^T q_t            (a decay per key channel from a
 //                              a_t = sigmoid(W2 u_t + b)^(1/tau)                                 low-rank projection, lowrank_decay_kernel)
 //
-//   gated delta rule:          S <- g_t S ;   S <- S + k_t (b_t (v_t - S^T k_t))^T ;   o_t = S^T q_t  (one decay g_t and one write strength b_t
-//                                                                                  per head and token; several heads may share q and k)
-//
 // (a step of single tokens: gla_token_kernel, the whole of it with the head's norm and gate)
 //
-// From the gated write on the state is [K, V] with V value channels that need not equal K; the first two have V = K.
+// In the last three the state is [K, V] with V value channels that need not equal K; the first two have V = K.
 //
 // A CTA per (request, head, 16 columns of S) walks the request's tokens of the step in order; column j of S (the K numbers
 // that meet value channel j) lives in the registers of eight neighbouring threads, so a token costs K/8 multiply-adds per
@@ -95,8 +92,7 @@ __device__ __forceinline__ void stage_async(float* dst, const float* src, int by
 
 // MODE 0: decay and bonus; MODE 1: generalized delta rule; MODE 2: gated write (no k: 1 - d stands for it; KV value
 // channels, the columns of S); MODE 3: retention (one decay per head); MODE 4: gated linear attention (KV value channels; what
-// comes out is multiplied by out_scale); MODE 5: gated delta rule (`share` heads read one head of r and k; bonus [T, N]: the write
-// strengths, inv [T, N]: the decays, both ready made).  d: the decays, a: the removal rates (MODE 1), both ready made
+// comes out is multiplied by out_scale).  d: the decays, a: the removal rates (MODE 1), both ready made
 // (scan_gates_kernel).  last_in (MODE 0, may be null): the mixer's input rows [T, W] of the activation type; the
 // request's last row is kept as fp32 at state + prev_off (the next step's "previous token").
 //
@@ -111,12 +107,12 @@ __global__ void __launch_bounds__(kScanThreads)
 state_scan_kernel(ScanInput r, ScanInput k, ScanInput v, ScanInput d, ScanInput a, const float* __restrict__ bonus,
                   const float* __restrict__ inv, float* __restrict__ state, long long state_stride, const int32_t* __restrict__ q_start,
                   const int32_t* __restrict__ slots, float* __restrict__ out, const TA* __restrict__ last_in, int W,
-                  long long prev_off, int N, int K, int KV, int vec, float out_scale, int share) {
+                  long long prev_off, int N, int K, int KV, int vec, float out_scale) {
     constexpr int RPT = KMAX / kSplit;                                  // rows of S per thread
     constexpr int kScanTokens = MODE == 4 && KMAX > 192 ? 4 : ::kScanTokens;   // (three vectors of 256 channels: four tokens fit 48 KB)
-    __shared__ __align__(16) float rs[2][kScanTokens][KMAX], ks[2][MODE == 2 ? 1 : kScanTokens][KMAX], ds[2][MODE == 3 || MODE == 5 ? 1 : kScanTokens][KMAX];
+    __shared__ __align__(16) float rs[2][kScanTokens][KMAX], ks[2][MODE == 2 ? 1 : kScanTokens][KMAX], ds[2][MODE == 3 ? 1 : kScanTokens][KMAX];
     __shared__ __align__(16) float as[2][MODE == 1 ? kScanTokens : 1][KMAX], vs[2][kScanTokens][kCols], us[KMAX];
-    __shared__ float is[2][kScanTokens], bs[2][kScanTokens];            // MODE 1: 1 / (|k|^2 + 1e-6) of the staged tokens; MODE 5: decays, strengths
+    __shared__ float is[2][kScanTokens];                                // MODE 1: 1 / (|k|^2 + 1e-6) of the staged tokens
     forge::pdl_launch_dependents();
     const int s = blockIdx.x, head = blockIdx.y, tid = threadIdx.x, jl = tid / kSplit, q = tid % kSplit;
     const int j = blockIdx.z * kCols + jl;
@@ -126,7 +122,7 @@ state_scan_kernel(ScanInput r, ScanInput k, ScanInput v, ScanInput d, ScanInput 
     for (int i = tid; i < 2 * kScanTokens * KMAX; i += kScanThreads) {
         (&rs[0][0][0])[i] = 0.f;
         if (MODE != 2) (&ks[0][0][0])[i] = 0.f;          // (mode 2 has no keys: its ks is a stub that nothing reads)
-        if (MODE != 3 && MODE != 5) (&ds[0][0][0])[i] = 0.f;          // (modes 3 and 5 have one decay per head: nothing staged)
+        if (MODE != 3) (&ds[0][0][0])[i] = 0.f;          // (mode 3 has one decay per head: nothing staged)
         if (MODE == 1) (&as[0][0][0])[i] = 0.f;
     }
     for (int i = tid; i < 2 * kScanTokens * kCols; i += kScanThreads) (&vs[0][0][0])[i] = 0.f;
@@ -142,21 +138,19 @@ state_scan_kernel(ScanInput r, ScanInput k, ScanInput v, ScanInput d, ScanInput 
     for (int ii = 0; ii < RPT; ++ii) S[ii] = (live && row_of(ii) < K) ? S_g[(size_t)row_of(ii) * KV + j] : 0.f;
 
     const int piece = vec ? 4 : 1, pieces = K / piece;                   // a staged vector in pieces of 16 or 4 bytes
-    const int head_qk = MODE == 5 ? head / share : head;                 // whose r and k this head reads
     auto fetch = [&](int buf, int tb) {
         const int n = min(kScanTokens, t_hi - tb);
         for (int p = tid; p < n * pieces; p += kScanThreads) {
             const int tt = p / pieces, ch = (p % pieces) * piece;
-            const size_t t = (size_t)(tb + tt), c = (size_t)head_qk * K + ch;
+            const size_t t = (size_t)(tb + tt), c = (size_t)head * K + ch;
             stage_async(&rs[buf][tt][ch], r.p + t * r.ld + c, piece * 4);
             if (MODE != 2) stage_async(&ks[buf][tt][ch], k.p + t * k.ld + c, piece * 4);
-            if (MODE != 3 && MODE != 5) stage_async(&ds[buf][tt][ch], d.p + t * d.ld + c, piece * 4);
+            if (MODE != 3) stage_async(&ds[buf][tt][ch], d.p + t * d.ld + c, piece * 4);
             if (MODE == 1) stage_async(&as[buf][tt][ch], a.p + t * a.ld + c, piece * 4);
         }
         const int tt = tid / kCols, jc = blockIdx.z * kCols + tid % kCols;              // values: this CTA's columns only
         if (tt < n && jc < KV) stage_async(&vs[buf][tt][tid % kCols], v.p + (size_t)(tb + tt) * v.ld + head * KV + jc, 4);
-        if ((MODE == 1 || MODE == 5) && tid < n) stage_async(&is[buf][tid], inv + (size_t)(tb + tid) * N + head, 4);
-        if (MODE == 5 && tid < n) stage_async(&bs[buf][tid], bonus + (size_t)(tb + tid) * N + head, 4);
+        if (MODE == 1 && tid < n) stage_async(&is[buf][tid], inv + (size_t)(tb + tid) * N + head, 4);
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     const float head_decay = MODE == 3 ? d.p[head] : 0.f;       // mode 3: d is one number per head
@@ -216,32 +210,6 @@ state_scan_kernel(ScanInput r, ScanInput k, ScanInput v, ScanInput d, ScanInput 
                     for (int e = 0; e < 4; ++e) {
                         const int ii = c4 * 4 + e;
                         S[ii] = fmaf(dv[e], S[ii], kv4[e] * vj);
-                        if (e & 1) acc1 = fmaf(rv[e], S[ii], acc1);
-                        else acc0 = fmaf(rv[e], S[ii], acc0);
-                    }
-                }
-            } else if (MODE == 5) {
-                float held0 = 0.f, held1 = 0.f, held2 = 0.f, held3 = 0.f;      // this thread's share of S^T k (its column)
-#pragma unroll
-                for (int c4 = 0; c4 < RPT / 4; ++c4) {
-                    const float4 kk = k4[c4 * kSplit];
-                    held0 = fmaf(kk.x, S[c4 * 4], held0);
-                    held1 = fmaf(kk.y, S[c4 * 4 + 1], held1);
-                    held2 = fmaf(kk.z, S[c4 * 4 + 2], held2);
-                    held3 = fmaf(kk.w, S[c4 * 4 + 3], held3);
-                }
-                float held = (held0 + held1) + (held2 + held3);
-#pragma unroll
-                for (int o = 1; o < kSplit; o <<= 1) held += __shfl_xor_sync(0xffffffffu, held, o);
-                const float g = is[buf][tt], u = bs[buf][tt] * fmaf(-g, held, vj);
-#pragma unroll
-                for (int c4 = 0; c4 < RPT / 4; ++c4) {
-                    const float4 rr = r4[c4 * kSplit], kk = k4[c4 * kSplit];
-                    const float rv[4] = {rr.x, rr.y, rr.z, rr.w}, kv4[4] = {kk.x, kk.y, kk.z, kk.w};
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) {
-                        const int ii = c4 * 4 + e;
-                        S[ii] = fmaf(g, S[ii], kv4[e] * u);
                         if (e & 1) acc1 = fmaf(rv[e], S[ii], acc1);
                         else acc0 = fmaf(rv[e], S[ii], acc0);
                     }
@@ -539,12 +507,12 @@ gla_token_kernel(ScanInput q, ScanInput k, ScanInput v, ScanInput g, ScanInput u
 template <int MODE, typename TA>
 cudaError_t launch_scan(int kmax, dim3 grid, cudaStream_t stream, ScanInput r, ScanInput k, ScanInput v, ScanInput d, ScanInput a,
                         const float* bonus, const float* inv, float* state, long long stride, const int32_t* q_start, const int32_t* slots,
-                        float* out, const TA* last_in, int W, long long prev_off, int N, int K, int KV, int vec, float out_scale = 1.0f, int share = 1) {
+                        float* out, const TA* last_in, int W, long long prev_off, int N, int K, int KV, int vec, float out_scale = 1.0f) {
 #define FORGE_SCAN_CASE(KM)                                                                                                  \
     case KM:                                                                                                                 \
         return forge::launch(state_scan_kernel<KM, MODE, TA>, grid, dim3(kScanThreads), 0, stream, 1, r, k, v, d, a, bonus, inv, state, \
-                             stride, q_start, slots, out, last_in, W, prev_off, N, K, KV, vec, out_scale, share);
-    if constexpr (MODE >= 2) {   // the gated write stages no keys, retention and the gated delta rule no decays: heads of up to 256 key channels fit
+                             stride, q_start, slots, out, last_in, W, prev_off, N, K, KV, vec, out_scale);
+    if constexpr (MODE >= 2) {   // the gated write stages no keys, retention no decays: heads of up to 256 key channels fit
         switch (kmax) {
             FORGE_SCAN_CASE(192) FORGE_SCAN_CASE(256)
             default: break;
@@ -666,48 +634,7 @@ extern "C" int forge_gla_scan(const float* q, int ld_q, const float* k, int ld_k
     return forge::check_launch("gla_scan", e);
 }
 
-extern "C" int forge_silu_columns(float* x, long long ld, int T, int n, cudaStream_t stream);       // recurrent_token.cu
-
-// Lightning attention over the step's tokens: fp32 rows of ld numbers [q: N*K | k: N*K | v: N*KV] from proj on pass silu IN PLACE, then
-// S <- decay[n] S + k v^T, out = S^T q per head (out fp32 [T, N*KV]; decay fp32 [N]; a head's state is [K, KV]): the scan of retention.
-extern "C" int forge_lightning_scan(float* proj, int ld, const float* decay, float* state, long long state_stride, const int32_t* q_start,
-                                    const int32_t* slots, float* out, int T, int S, int N, int K, int KV, cudaStream_t stream) {
-    if (T < 0 || S < 0 || N <= 0 || K <= 0 || KV <= 0 || ld < N * (2 * K + KV)) return forge::fail(FORGE_ERR_ARG, "lightning_scan: bad sizes S=%d N=%d K=%d V=%d ld=%d", S, N, K, KV, ld);
-    if (K > 256) return forge::fail(FORGE_ERR_UNSUPPORTED, "lightning_scan: heads of %d key channels (at most 256)", K);
-    if (state_stride < (long long)N * K * KV) return forge::fail(FORGE_ERR_ARG, "lightning_scan: state rows are too short");
-    if (S == 0 || T == 0) return FORGE_OK;
-    const int rc = forge_silu_columns(proj, ld, T, N * (2 * K + KV), stream);
-    if (rc != FORGE_OK) return rc;
-    const int kmax = K <= 128 ? (K + 31) / 32 * 32 : (K <= 192 ? 192 : 256);
-    ScanInput Q{proj, ld}, Kk{proj + N * K, ld}, V{proj + 2 * N * K, ld}, D{decay, 0};
-    const int vec = (K % 4 == 0 && ((uintptr_t)proj & 15) == 0 && ld % 4 == 0) ? 1 : 0;
-    cudaError_t e = launch_scan<3, float>(kmax, dim3(S, N, (KV + kCols - 1) / kCols), stream, Q, Kk, V, D, D, nullptr, nullptr, state, state_stride,
-                                          q_start, slots, out, nullptr, 0, 0, N, K, KV, vec);
-    return forge::check_launch("lightning_scan", e);
-}
-
-// Gated delta rule over the step's tokens: per head n, with q and k of head n / (N / M),
-//     S <- g S;   S <- S + k (beta (v - S^T k))^T;   out = S^T q.
-// q, k fp32 (row t at p + t * ld, M heads of K channels), v fp32 (N heads of KV channels), g and beta fp32 [T, N]; out fp32 [T, N*KV]; a
-// head's state is [K, KV], row slots[s] of `state` holds request s's N of them from its start.
-extern "C" int forge_gated_delta_scan(const float* q, int ld_q, const float* k, int ld_k, const float* v, int ld_v, const float* g,
-                                      const float* beta, float* state, long long state_stride, const int32_t* q_start, const int32_t* slots,
-                                      float* out, int T, int S, int N, int M, int K, int KV, cudaStream_t stream) {
-    if (T < 0 || S < 0 || N <= 0 || M <= 0 || N % M != 0 || K <= 0 || KV <= 0) return forge::fail(FORGE_ERR_ARG, "gated_delta_scan: bad sizes S=%d N=%d M=%d K=%d V=%d", S, N, M, K, KV);
-    if (K > 256) return forge::fail(FORGE_ERR_UNSUPPORTED, "gated_delta_scan: heads of %d key channels (at most 256)", K);
-    if (state_stride < (long long)N * K * KV) return forge::fail(FORGE_ERR_ARG, "gated_delta_scan: state rows are too short");
-    if (S == 0 || T == 0) return FORGE_OK;
-    const int kmax = K <= 128 ? (K + 31) / 32 * 32 : (K <= 192 ? 192 : 256);
-    const dim3 grid(S, N, (KV + kCols - 1) / kCols);
-    ScanInput Q{q, ld_q}, Kk{k, ld_k}, V{v, ld_v};
-    auto aligned = [](const float* p, int ld) { return ((uintptr_t)p & 15) == 0 && ld % 4 == 0; };
-    const int vec = (K % 4 == 0 && aligned(q, ld_q) && aligned(k, ld_k)) ? 1 : 0;
-    cudaError_t e = launch_scan<5, float>(kmax, grid, stream, Q, Kk, V, Q, Q, beta, g, state, state_stride, q_start, slots, out, nullptr, 0, 0, N, K,
-                                          KV, vec, 1.0f, N / M);
-    return forge::check_launch("gated_delta_scan", e);
-}
-
-// forge_gla_scan for a step in which every request brings one token (S tokens, request s's is token q_start[s]), with the head's norm
+// The same for a step in which every request brings one token (S tokens, request s's is token q_start[s]), with the head's norm
 // (weight fp32 [KV], eps), and silu of the gate g (fp32 rows, N*KV columns) multiplied on; out of out_dtype, rows of out_ld with the
 // N*KV values at their start.
 extern "C" int forge_gla_token(const float* q, int ld_q, const float* k, int ld_k, const float* v, int ld_v, const float* g, int ld_g,

@@ -29,22 +29,36 @@ __device__ __forceinline__ float softplusf(float x) { return fmaxf(x, 0.f) + log
 __device__ __forceinline__ float decayf(float x) { return 1.0f + expm1f(-x); }
 
 struct ShortConv {
-    const float* w;                   // fp32 [channels, taps], the last column is the current token's; null: no convolution
+    const float* w;                   // fp32 [taps, channels], row 0 the current token's, row j that of the token j before it
     int taps;
     int channels;                     // numbers in a row of the ring (all tensors that are convolved, side by side)
 };
 
-// The convolution of channel c (its weight row and its place in the ring) of token t at position pos; x: the channel's numbers in the
-// projection; `first`: the request's first token of the step; ring: the request's ring.
+constexpr int kTaps = 8;              // taps whose inputs and weights are all asked for before the first is used
+
+// The convolution of channel c (its column of w and its place in the ring) of token t at position pos; x: the channel's numbers in the
+// projection; `first`: the request's first token of the step; ring: the request's ring.  The oldest input is added first, whatever the cut.
 __device__ __forceinline__ float convolve(const ShortConv& cv, const float* __restrict__ x, int ld, int t, int first, int pos, int c,
                                           const float* __restrict__ ring) {
-    const float* w = cv.w + (size_t)c * cv.taps;
+    const int at = pos % cv.taps;
+    auto input = [&](int j) {
+        if (t - j >= first) return x[(size_t)(t - j) * ld];
+        return ring[(size_t)(at >= j ? at - j : at - j + cv.taps) * cv.channels + c];
+    };
     float a = 0.f;
-    for (int j = cv.taps - 1; j >= 0; --j) {             // the oldest input first, whatever the step's cut
-        if (pos < j) continue;
-        const float v = t - j >= first ? x[(size_t)(t - j) * ld] : ring[(size_t)((pos - j) % cv.taps) * cv.channels + c];
-        a = fmaf(w[cv.taps - 1 - j], v, a);
+    for (int j = cv.taps - 1; j >= kTaps; --j)
+        if (pos >= j) a = fmaf(cv.w[(size_t)j * cv.channels + c], input(j), a);
+    float v[kTaps], w[kTaps];
+#pragma unroll
+    for (int j = 0; j < kTaps; ++j) {
+        v[j] = w[j] = 0.f;
+        if (j < cv.taps && pos >= j) {
+            v[j] = input(j);
+            w[j] = cv.w[(size_t)j * cv.channels + c];
+        }
     }
+#pragma unroll
+    for (int j = kTaps - 1; j >= 0; --j) a = fmaf(w[j], v[j], a);
     return a;
 }
 
@@ -63,40 +77,104 @@ struct DeltaPrepare {
 };
 
 constexpr int kUnitRegs = 8;          // channels of a q or k head that a lane holds (heads of up to 256)
+constexpr int kPrepTokens = 4;        // consecutive tokens that a warp takes at a time, so that most inputs are read once
+constexpr int kPrepTiles = 4;         // such tiles that a warp takes one after the other
 
-// A warp per (token, head of q, k or v); the four warps of a CTA take four consecutive tokens, which share most of their inputs.
-__global__ void __launch_bounds__(128)
-delta_prepare_kernel(const DeltaPrepare d) {
-    forge::pdl_wait();
-    const int t = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31, unit = blockIdx.y;
-    if (t >= d.T) return;
-    const int s = d.tok_req[t], first = d.q_start[s], pos = d.positions[t], C = 2 * d.M * d.K + d.N * d.V;
-    const float* ring = d.state + (size_t)d.slots[s] * d.stride + d.ring_off;
+// kPrepTokens neighbouring tokens of one channel, t0 the first.  inner: all of them and all that they look back on are one request's
+// tokens of this step (and n == kPrepTokens, taps <= kTaps); then a window of inputs is read once and slides over the taps.
+__device__ __forceinline__ void convolve_tile(const DeltaPrepare& d, const float* __restrict__ x, int c, int t0, int n, bool inner, float (&y)[kPrepTokens]) {
+    if (inner) {
+        float v[kTaps - 1 + kPrepTokens], w[kTaps];
+#pragma unroll
+        for (int i = 0; i < kTaps - 1 + kPrepTokens; ++i) {               // v[i]: token t0 + i - (kTaps - 1)
+            const int back = kTaps - 1 - i;
+            v[i] = back < d.cv.taps ? x[(ptrdiff_t)(t0 - back) * d.p.ld] : 0.f;
+        }
+#pragma unroll
+        for (int j = 0; j < kTaps; ++j) w[j] = j < d.cv.taps ? d.cv.w[(size_t)j * d.cv.channels + c] : 0.f;
+#pragma unroll
+        for (int k = 0; k < kPrepTokens; ++k) {
+            float a = 0.f;
+#pragma unroll
+            for (int j = kTaps - 1; j >= 0; --j) a = fmaf(w[j], v[kTaps - 1 + k - j], a);
+            y[k] = siluf(a);
+        }
+        return;
+    }
+    for (int k = 0; k < kPrepTokens; ++k) {
+        y[k] = 0.f;
+        if (k >= n) continue;
+        const int t = t0 + k, s = d.tok_req[t];
+        y[k] = siluf(convolve(d.cv, x, d.p.ld, t, d.q_start[s], d.positions[t], c, d.state + (size_t)d.slots[s] * d.stride + d.ring_off));
+    }
+}
+
+// One tile of one head of q, k or v, by a warp.  NC: the lanes' channels of a q or k head.
+template <int NC>
+__device__ __forceinline__ void prepare_tile(const DeltaPrepare& d, int t0, int n, bool inner, int unit, int lane) {
+    const int C = 2 * d.M * d.K + d.N * d.V;
     if (unit < 2 * d.M) {
         const int c0 = unit * d.K;
-        float x[kUnitRegs], ss = 0.f;
+        float x[NC][kPrepTokens], ss[kPrepTokens];
 #pragma unroll
-        for (int i = 0; i < kUnitRegs; ++i) {
+        for (int k = 0; k < kPrepTokens; ++k) ss[k] = 0.f;
+#pragma unroll
+        for (int i = 0; i < NC; ++i) {
             const int c = lane + 32 * i;
-            x[i] = c < d.K ? siluf(convolve(d.cv, d.p.p + c0 + c, d.p.ld, t, first, pos, c0 + c, ring)) : 0.f;
-            ss = fmaf(x[i], x[i], ss);
+            if (32 * i >= d.K) continue;                                  // (the same for the whole warp)
+            if (c < d.K) convolve_tile(d, d.p.p + c0 + c, c0 + c, t0, n, inner, x[i]);
+#pragma unroll
+            for (int k = 0; k < kPrepTokens; ++k) {
+                if (c >= d.K) x[i][k] = 0.f;
+                ss[k] = fmaf(x[i][k], x[i][k], ss[k]);
+            }
         }
-        float inv = 1.0f / sqrtf(forge::warp_sum(ss) + 1e-6f);
-        if (unit < d.M) inv *= 1.0f / sqrtf((float)d.K);
+        const float scale = unit < d.M ? 1.0f / sqrtf((float)d.K) : 1.0f;
 #pragma unroll
-        for (int i = 0; i < kUnitRegs; ++i) {
-            const int c = lane + 32 * i;
-            if (c < d.K) d.qkv[(size_t)t * C + c0 + c] = x[i] * inv;
+        for (int k = 0; k < kPrepTokens; ++k) {
+            const float inv = scale / sqrtf(forge::warp_sum(ss[k]) + 1e-6f);
+            if (k >= n) continue;
+#pragma unroll
+            for (int i = 0; i < NC; ++i) {
+                const int c = lane + 32 * i;
+                if (c < d.K) d.qkv[(size_t)(t0 + k) * C + c0 + c] = x[i][k] * inv;
+            }
         }
         return;
     }
     const int head = unit - 2 * d.M, c0 = 2 * d.M * d.K + head * d.V;
-    for (int c = lane; c < d.V; c += 32)
-        d.qkv[(size_t)t * C + c0 + c] = siluf(convolve(d.cv, d.p.p + c0 + c, d.p.ld, t, first, pos, c0 + c, ring));
-    if (lane == 0) {
-        const float* row = d.p.p + (size_t)t * d.p.ld;
-        d.beta[(size_t)t * d.N + head] = sigmoidf(row[d.b_col + head]);
-        d.g[(size_t)t * d.N + head] = decayf(d.decay_rate[head] * softplusf(row[d.a_col + head] + d.dt[head]));
+    for (int c = lane; c < d.V; c += 32) {
+        float y[kPrepTokens];
+        convolve_tile(d, d.p.p + c0 + c, c0 + c, t0, n, inner, y);
+#pragma unroll
+        for (int k = 0; k < kPrepTokens; ++k)
+            if (k < n) d.qkv[(size_t)(t0 + k) * C + c0 + c] = y[k];
+    }
+    if (lane < n) {
+        const float* row = d.p.p + (size_t)(t0 + lane) * d.p.ld;
+        d.beta[(size_t)(t0 + lane) * d.N + head] = sigmoidf(row[d.b_col + head]);
+        d.g[(size_t)(t0 + lane) * d.N + head] = decayf(d.decay_rate[head] * softplusf(row[d.a_col + head] + d.dt[head]));
+    }
+}
+
+// A warp per (kPrepTiles tiles of kPrepTokens tokens, head of q, k or v).
+template <int NC>
+__global__ void __launch_bounds__(128, NC <= 4 ? 6 : 4)
+delta_prepare_kernel(const DeltaPrepare d) {
+    forge::pdl_wait();
+    const int first = (blockIdx.x * 4 + (threadIdx.x >> 5)) * kPrepTokens * kPrepTiles, lane = threadIdx.x & 31;
+    if (first >= d.T) return;
+    const int last = min(first + kPrepTokens * kPrepTiles, d.T) - 1, s0 = d.tok_req[first], back = d.cv.taps - 1;
+    const bool one = d.cv.taps <= kTaps && d.tok_req[last] == s0 && first - back >= d.q_start[s0];
+#pragma unroll 1
+    for (int t0 = first; t0 <= last; t0 += kPrepTokens) {
+        const int n = min(kPrepTokens, d.T - t0);
+        bool inner = one;
+        if (!one && d.cv.taps <= kTaps) {
+            const int s = d.tok_req[t0];
+            inner = d.tok_req[t0 + n - 1] == s && t0 - back >= d.q_start[s];
+        }
+        prepare_tile<NC>(d, t0, n, inner && n == kPrepTokens, blockIdx.y, lane);
     }
 }
 
@@ -178,7 +256,7 @@ gated_rows_kernel(const float* __restrict__ o, const float* __restrict__ w, Colu
 }
 
 constexpr int kTokenThreads = 512;        // at most
-constexpr int kHeld = 16;                 // packs of the state that a thread holds
+constexpr int kHeld = 16;                 // packs of the state that a thread holds, at most
 
 struct TokenState {
     Columns q, k, v;                  // before convolution and activation
@@ -199,20 +277,21 @@ struct TokenState {
 // at the state to the write (longer heads read theirs again).  DELTA: one look gives S^T k and S^T q at once, the RG partial sums are
 // added in a fixed order, and with u = beta (v - g S^T k) the output is g S^T q + (k . q) u.  Else S <- decay S + k v^T, o = S^T q.
 // out: DELTA: the normed and gated heads in the activation type; else the heads as they are, fp32.
-template <int P, bool DELTA, typename TA>
-__global__ void __launch_bounds__(kTokenThreads)
+// kMost: the most threads of a launch, kCtas: how many such CTAs an SM should hold.
+template <int P, int kHeld, int kMost, int kCtas, bool DELTA, typename TA>
+__global__ void __launch_bounds__(kMost, kCtas)
 token_state_kernel(const TokenState d, TA* __restrict__ out, long long out_ld) {
     using S4 = typename Pack<P>::type;
     extern __shared__ __align__(16) float sm[];
-    __shared__ float red[3][32];
+    __shared__ float red[32];
     const int K = d.K, V = d.V, CG = d.CG, RG = d.RG;
-    float* qs = sm;                    // [K]
+    float* qs = sm;                    // [K] q, k and v after convolution and silu, side by side
     float* ks = qs + K;                // [K]
     float* vs = ks + K;                // [V]
     float* part = vs + V;              // [RG][V] partial sums of S^T q; DELTA: then [RG][V] of S^T k
     forge::pdl_launch_dependents();
     forge::pdl_wait();
-    const int threads = blockDim.x, s = blockIdx.x, head = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int threads = blockDim.x, s = blockIdx.x, head = blockIdx.y, tid = threadIdx.x, lane = tid & 31;
     const int t = d.q_start[s], share = d.N / d.M, hk = head / share;
     float* row_of_slot = d.state + (size_t)d.slots[s] * d.stride;
     float* S = row_of_slot + (size_t)head * K * V;
@@ -225,36 +304,29 @@ token_state_kernel(const TokenState d, TA* __restrict__ out, long long out_ld) {
         const int row = rg + m * RG;
         if (live && row < K) held[m] = reinterpret_cast<const S4*>(S + (size_t)row * V)[cp];
     }
-    float g = 0.f, beta = 0.f, qq = 0.f, kk = 0.f, qk = 0.f;
+    float g = 0.f, beta = 0.f, gate[P], weight[P];
     if (DELTA) {
-        const int pos = d.positions[t], at = pos % d.cv.taps;
-        float* ring = row_of_slot + d.ring_off;
-        float* now = ring + (size_t)at * d.cv.channels;
-        for (int i = tid; i < K; i += threads) {
-            const int cq = hk * K + i, ck = d.M * K + cq;
-            const float x = siluf(convolve(d.cv, d.q.p + cq, d.q.ld, t, t, pos, cq, ring));
-            const float y = siluf(convolve(d.cv, d.k.p + cq, d.k.ld, t, t, pos, ck, ring));
-            qs[i] = x;
-            ks[i] = y;
-            qq = fmaf(x, x, qq);
-            kk = fmaf(y, y, kk);
-            qk = fmaf(x, y, qk);
-            if (head % share == 0) {                       // the token's own row of the ring, which nobody reads in this step
-                now[cq] = d.q.p[(size_t)t * d.q.ld + cq];
-                now[ck] = d.k.p[(size_t)t * d.k.ld + cq];
+        const float a_in = d.a.p[(size_t)t * d.a.ld + head] + d.dt[head], b_in = d.b.p[(size_t)t * d.b.ld + head], rate = d.decay[head];
+        if (rg == 0) {                                     // what the end needs is asked for now
+#pragma unroll
+            for (int e = 0; e < P; ++e) {
+                weight[e] = d.weight[cp * P + e];
+                gate[e] = d.gate.p[(size_t)t * d.gate.ld + (size_t)head * V + cp * P + e];
             }
         }
-        for (int i = tid; i < V; i += threads) {
-            const int c = head * V + i, cc = 2 * d.M * K + c;
-            vs[i] = siluf(convolve(d.cv, d.v.p + c, d.v.ld, t, t, pos, cc, ring));
-            now[cc] = d.v.p[(size_t)t * d.v.ld + c];
+        const int pos = d.positions[t];
+        float* ring = row_of_slot + d.ring_off;
+        float* now = ring + (size_t)(pos % d.cv.taps) * d.cv.channels;
+#pragma unroll 2
+        for (int i = tid; i < 2 * K + V; i += threads) {
+            // q and k of the shared head, then the head's values: column of the projection's [q | k | v] and of the ring
+            const int c = i < K ? hk * K + i : (i < 2 * K ? (d.M - 1 + hk) * K + i : 2 * (d.M - 1) * K + head * V + i);
+            sm[i] = siluf(convolve(d.cv, d.q.p + c, d.q.ld, t, t, pos, c, ring));
+            // the token's own row of the ring, which nobody reads in this step
+            if (i >= 2 * K || head % share == 0) now[c] = d.q.p[(size_t)t * d.q.ld + c];
         }
-        g = decayf(d.decay[head] * softplusf(d.a.p[(size_t)t * d.a.ld + head] + d.dt[head]));
-        beta = sigmoidf(d.b.p[(size_t)t * d.b.ld + head]);
-        qq = forge::warp_sum(qq);
-        kk = forge::warp_sum(kk);
-        qk = forge::warp_sum(qk);
-        if (lane == 0) { red[0][warp] = qq; red[1][warp] = kk; red[2][warp] = qk; }
+        g = decayf(rate * softplusf(a_in));
+        beta = sigmoidf(b_in);
     } else {
         g = d.decay[head];
         for (int i = tid; i < K; i += threads) {
@@ -266,8 +338,15 @@ token_state_kernel(const TokenState d, TA* __restrict__ out, long long out_ld) {
     __syncthreads();
     float kscale = 1.f;
     if (DELTA) {
-        qq = kk = qk = 0.f;
-        for (int i = 0; i < (threads + 31) / 32; ++i) { qq += red[0][i]; kk += red[1][i]; qk += red[2][i]; }
+        float qq = 0.f, kk = 0.f, qk = 0.f;                // every warp for itself
+        for (int i = lane; i < K; i += 32) {
+            qq = fmaf(qs[i], qs[i], qq);
+            kk = fmaf(ks[i], ks[i], kk);
+            qk = fmaf(qs[i], ks[i], qk);
+        }
+        qq = forge::warp_sum(qq);
+        kk = forge::warp_sum(kk);
+        qk = forge::warp_sum(qk);
         const float qscale = 1.0f / (sqrtf(qq + 1e-6f) * sqrtf((float)K));
         kscale = 1.0f / sqrtf(kk + 1e-6f);
         qk *= qscale * kscale;
@@ -286,6 +365,7 @@ token_state_kernel(const TokenState d, TA* __restrict__ out, long long out_ld) {
 #pragma unroll
             for (int m = 0; m < kHeld; ++m)
                 if (rg + m * RG < K) look(rg + m * RG, held[m]);
+#pragma unroll 1
             for (int row = rg + kHeld * RG; row < K; row += RG) look(row, reinterpret_cast<const S4*>(S + (size_t)row * V)[cp]);
             reinterpret_cast<S4*>(part + (size_t)rg * V)[cp] = aq;
             reinterpret_cast<S4*>(part + (size_t)(RG + rg) * V)[cp] = ak;
@@ -318,16 +398,16 @@ token_state_kernel(const TokenState d, TA* __restrict__ out, long long out_ld) {
 #pragma unroll
             for (int m = 0; m < kHeld; ++m)
                 if (rg + m * RG < K) write(rg + m * RG, held[m]);
+#pragma unroll 1
             for (int row = rg + kHeld * RG; row < K; row += RG) write(row, reinterpret_cast<const S4*>(S + (size_t)row * V)[cp]);
         }
         // the head's norm: the first CG threads have every output once
-        const float inv = 1.0f / sqrtf(forge::block_sum(rg == 0 ? ss : 0.f, red[0]) / (float)V + d.eps);
+        const float inv = 1.0f / sqrtf(forge::block_sum(rg == 0 ? ss : 0.f, red) / (float)V + d.eps);
         if (rg == 0) {
 #pragma unroll
             for (int e = 0; e < P; ++e) {
                 const int c = cp * P + e;
-                out[(size_t)t * out_ld + (size_t)head * V + c] =
-                    forge::from_float<TA>(o[e] * inv * d.weight[c] * siluf(d.gate.p[(size_t)t * d.gate.ld + (size_t)head * V + c]));
+                out[(size_t)t * out_ld + (size_t)head * V + c] = forge::from_float<TA>(o[e] * inv * weight[e] * siluf(gate[e]));
             }
         }
     } else {
@@ -347,6 +427,7 @@ token_state_kernel(const TokenState d, TA* __restrict__ out, long long out_ld) {
 #pragma unroll
             for (int m = 0; m < kHeld; ++m)
                 if (rg + m * RG < K) step(rg + m * RG, held[m]);
+#pragma unroll 1
             for (int row = rg + kHeld * RG; row < K; row += RG) step(row, reinterpret_cast<const S4*>(S + (size_t)row * V)[cp]);
             reinterpret_cast<S4*>(part + (size_t)rg * V)[cp] = acc;
         }
@@ -385,10 +466,18 @@ bool token_vec(const void* state, long long stride, int K, int V) {
     return V % 4 == 0 && K % 2 == 0 && stride % 4 == 0 && ((uintptr_t)state & 15) == 0;
 }
 
+template <bool DELTA, typename TO>
+cudaError_t launch_token(bool vec, const TokenShape& sh, dim3 grid, cudaStream_t stream, const TokenState& d, TO* out, long long out_ld) {
+    const bool few = (d.K + sh.RG - 1) / sh.RG <= kHeld / 2;            // rows a thread holds: half the registers where half are enough
+    auto kernel = vec ? (few && sh.threads == 128 ? token_state_kernel<4, kHeld / 2, 128, 5, DELTA, TO> : token_state_kernel<4, kHeld, kTokenThreads, 1, DELTA, TO>)
+                      : (few ? token_state_kernel<1, kHeld / 2, kTokenThreads, 1, DELTA, TO> : token_state_kernel<1, kHeld, kTokenThreads, 1, DELTA, TO>);
+    return forge::launch(kernel, grid, dim3(sh.threads), sh.smem, stream, 1, d, out, out_ld);
+}
+
 }  // namespace
 
 // proj fp32 rows of ld numbers: [q: M*K | k: M*K | v: N*V] from their start, then b and a (N each) from columns b_col and a_col.
-// conv_w fp32 [2*M*K + N*V, taps].  state fp32 rows of `stride` numbers, row slots[s] holds request s's ring [taps, 2*M*K + N*V] from
+// conv_w fp32 [taps, 2*M*K + N*V], row j the weights of the token j before.  state fp32 rows of `stride` numbers, row slots[s] holds request s's ring [taps, 2*M*K + N*V] from
 // ring_off on.  Leaves qkv fp32 [T, 2*M*K + N*V], g and beta fp32 [T, N], and the rings as they are after the step.
 extern "C" int forge_delta_prepare(const float* proj, int ld, int b_col, int a_col, const float* conv_w, int taps, float* state, long long stride,
                                    long long ring_off, const int32_t* tok_req, const int32_t* q_start, const int32_t* positions,
@@ -403,7 +492,9 @@ extern "C" int forge_delta_prepare(const float* proj, int ld, int b_col, int a_c
     if (T == 0 || S == 0) return FORGE_OK;
     const ShortConv cv{conv_w, taps, (int)C};
     const DeltaPrepare d{{proj, ld}, b_col, a_col, cv, state, stride, ring_off, tok_req, q_start, positions, slots, decay_rate, dt, qkv, g, beta, T, N, M, K, V};
-    cudaError_t e = forge::launch(delta_prepare_kernel, dim3((T + 3) / 4, 2 * M + N), dim3(128), 0, stream, 1, d);
+    constexpr int per_cta = 4 * kPrepTokens * kPrepTiles;
+    cudaError_t e = forge::launch(K <= 64 ? delta_prepare_kernel<2> : K <= 128 ? delta_prepare_kernel<4> : delta_prepare_kernel<kUnitRegs>,
+                                  dim3((T + per_cta - 1) / per_cta, 2 * M + N), dim3(128), 0, stream, 1, d);
     if (e != cudaSuccess) return forge::check_launch("delta_prepare", e);
     e = forge::launch(conv_keep_kernel, dim3(S, (unsigned)((C + 255) / 256)), dim3(256), 0, stream, 1, Columns{proj, ld}, cv, state, stride, ring_off,
                       q_start, positions, slots);
@@ -459,8 +550,7 @@ extern "C" int forge_gated_delta_token(const float* proj, int ld, int g_col, int
                        decay_rate, dt, state, stride, ring_off, q_start, positions, slots, weight, eps, N, M, K, V, sh.CG, sh.RG};
     cudaError_t e = cudaSuccess;
     FORGE_DISPATCH_DTYPE(dtype, TO,
-        e = vec ? forge::launch(token_state_kernel<4, true, TO>, dim3(S, N), dim3(sh.threads), sh.smem, stream, 1, d, (TO*)out, out_ld)
-                : forge::launch(token_state_kernel<1, true, TO>, dim3(S, N), dim3(sh.threads), sh.smem, stream, 1, d, (TO*)out, out_ld));
+        e = launch_token<true>(vec, sh, dim3(S, N), stream, d, (TO*)out, out_ld));
     return forge::check_launch("gated_delta_token", e);
 }
 
@@ -476,7 +566,5 @@ extern "C" int forge_lightning_token(const float* proj, int ld, const float* dec
     if (S == 0) return FORGE_OK;
     const TokenState d{{proj, ld}, {proj + N * K, ld}, {proj + 2 * N * K, ld}, {nullptr, 1, 0}, {nullptr, 0}, {nullptr, 0}, {nullptr, 0},
                        decay, nullptr, state, stride, 0, q_start, nullptr, slots, nullptr, 0.f, N, N, K, V, sh.CG, sh.RG};
-    cudaError_t e = vec ? forge::launch(token_state_kernel<4, false, float>, dim3(S, N), dim3(sh.threads), sh.smem, stream, 1, d, out, (long long)N * V)
-                        : forge::launch(token_state_kernel<1, false, float>, dim3(S, N), dim3(sh.threads), sh.smem, stream, 1, d, out, (long long)N * V);
-    return forge::check_launch("lightning_token", e);
+    return forge::check_launch("lightning_token", launch_token<false>(vec, sh, dim3(S, N), stream, d, out, (long long)N * V));
 }

@@ -83,9 +83,9 @@ _SIGNATURES = {
         "forge_tanh_rows": [_P, _I, _P, _I, _I, _I, _P],
         "forge_gla_scan": [_P, _I] * 4 + [_I, _P, _P, _F, _F, _P, _P, _LL, _P, _P, _P, _I, _I, _I, _I, _I, _P],
         "forge_gla_token": [_P, _I] * 5 + [_I, _P, _P, _F, _F, _P, _LL, _P, _P, _P, _F, _P, _I, _LL, _I, _I, _I, _I, _P],
-        "forge_lightning_scan": [_P, _I, _P, _P, _LL, _P, _P, _P] + [_I] * 5 + [_P],
+        "forge_lightning_scan": [_P, _I, _P, _P, _P, _LL, _P, _P, _P] + [_I] * 5 + [_P],
         "forge_lightning_token": [_P, _I, _P, _P, _LL, _P, _P, _P] + [_I] * 4 + [_P],
-        "forge_gated_delta_scan": [_P, _I] * 3 + [_P, _P, _P, _LL, _P, _P, _P] + [_I] * 6 + [_P],
+        "forge_gated_delta_scan": [_P, _I] * 3 + [_P, _P, _P, _P, _LL, _P, _P, _P] + [_I] * 6 + [_P],
         "forge_delta_prepare": [_P, _I, _I, _I, _P, _I, _P, _LL, _LL] + [_P] * 9 + [_I] * 6 + [_P],
         "forge_gated_delta_token": [_P, _I, _I, _I, _I, _P, _I, _P, _LL, _LL] + [_P] * 6 + [_F, _P, _I, _LL] + [_I] * 5 + [_P],
         "forge_token_state_supports": [_I] * 3,
@@ -1234,7 +1234,13 @@ def gla_token(q, k, v, gate, hidden, rank, w2t, bias, tau, batch, state, N, K, K
     return out
 
 
-# a recurrence whose inputs pass silu, or a short convolution and silu, first (csrc/recurrent_token.cu)
+# recurrences whose inputs pass silu, or a short convolution and silu, first (csrc/recurrent_token.cu), eight tokens at a time
+# (csrc/recurrent_block.cu)
+
+def _gram(batch, T, heads, device):
+    """Room for the products of a block's keys with its keys and queries, for every head of keys and every block of every request."""
+    return new_tensor(((T // 8 + batch.num_requests) * heads * 64,), torch.float32, device)
+
 
 def token_state_supports(batch, K, V, delta):
     """A step in which every request brings one token, and heads of K x V numbers that the kernel of single tokens takes."""
@@ -1248,10 +1254,10 @@ def lightning_scan(proj, col, decay, batch, state, N, K, V):
     T = proj.shape[0]
     out = new_tensor((T, N * V), torch.float32, proj.device)
     p, ld = _cols(proj, col)
-    _check(lib, lib.forge_lightning_scan(p, ld, _need(decay, "decay", torch.float32), _need(state, "state", torch.float32, 2), state.shape[1],
+    _check(lib, lib.forge_lightning_scan(p, ld, _need(decay, "decay", torch.float32), _need(_gram(batch, T, N, proj.device), "gram"), _need(state, "state", torch.float32, 2), state.shape[1],
                                          _need(batch.q_start, "q_start", torch.int32), _need(batch.slots, "slots", torch.int32),
                                          _need(out, "out", torch.float32), T, batch.num_requests, N, K, V, _stream()), "lightning_scan")
-    count_launches(1)              # the kernel that applies silu
+    count_launches(2)              # the kernels that apply silu and take the blocks' products
     return out
 
 
@@ -1285,17 +1291,17 @@ def gated_rows(o, weight, gate, eps, out_dtype, out=None):
 
 def _delta_state(conv_w, state, N, M, K, V):
     """(taps, first number of the ring in a state row) of the gated delta rule's state; checks the sizes."""
-    C, taps = 2 * M * K + N * V, conv_w.shape[1]
+    C, taps = 2 * M * K + N * V, conv_w.shape[0]
     ring_off = N * K * V
-    if conv_w.shape[0] != C or state.shape[1] < ring_off + taps * C:
+    if conv_w.shape[1] != C or state.shape[1] < ring_off + taps * C:
         raise KernelError(f"gated delta rule: convolutions {tuple(conv_w.shape)} and state rows of {state.shape[1]} do not fit {N}/{M} heads of {K} x {V}")
     return taps, ring_off
 
 
 def gated_delta_prepare(proj, col, b_col, a_col, conv_w, decay_rate, dt, batch, state, N, M, K, V):
     """proj fp32 [T, ..]: [q: M*K | k: M*K | v: N*V] from column ``col``, and from ``b_col`` and ``a_col`` on the N inputs each of the write
-    strengths and the decays.  Convolves q, k, v over time (``conv_w`` fp32 [2*M*K + N*V, taps]; earlier inputs from the ring in the
-    request's ``state`` row behind its N*K*V numbers, which is brought up to date), silu, q and k to unit vectors, q times K^-1/2.
+    strengths and the decays.  Convolves q, k, v over time (``conv_w`` fp32 [taps, 2*M*K + N*V], row j the weights of the token
+    j before; earlier inputs from the ring in the request's ``state`` row behind its N*K*V numbers, which is brought up to date), silu, q and k to unit vectors, q times K^-1/2.
     Returns (qkv fp32 [T, 2*M*K + N*V], decays fp32 [T, N], strengths fp32 [T, N])."""
     lib = library("mixers")
     T = proj.shape[0]
@@ -1321,9 +1327,10 @@ def gated_delta_scan(qkv, g, beta, batch, state, N, M, K, V):
     out = new_tensor((T, N * V), torch.float32, qkv.device)
     (qp, ld), (kp, _), (vp, _) = _cols(qkv, 0), _cols(qkv, M * K), _cols(qkv, 2 * M * K)
     _check(lib, lib.forge_gated_delta_scan(
-        qp, ld, kp, ld, vp, ld, _need(g, "g", torch.float32, 2), _need(beta, "beta", torch.float32, 2), _need(state, "state", torch.float32, 2),
-        state.shape[1], _need(batch.q_start, "q_start", torch.int32), _need(batch.slots, "slots", torch.int32), _need(out, "out", torch.float32),
+        qp, ld, kp, ld, vp, ld, _need(g, "g", torch.float32, 2), _need(beta, "beta", torch.float32, 2), _need(_gram(batch, T, M, qkv.device), "gram"),
+        _need(state, "state", torch.float32, 2), state.shape[1], _need(batch.q_start, "q_start", torch.int32), _need(batch.slots, "slots", torch.int32), _need(out, "out", torch.float32),
         T, batch.num_requests, N, M, K, V, _stream()), "gated_delta_scan")
+    count_launches(1)              # the kernel that takes the blocks' products
     return out
 
 

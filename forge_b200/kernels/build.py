@@ -33,7 +33,7 @@ LIBRARIES = {
     # attention whose heads exchange weights, over a window with kept first tokens; attention with shaped scores (two maps per
     # head, a distance term); mixers with a matrix of state per head
     "mixers": ["attention_headmix.cu", "attention_headmix_mma.cu", "attention_scored.cu", "attention_scored_mma.cu", "recurrent.cu",
-               "recurrent_token.cu"],
+               "recurrent_token.cu", "recurrent_block.cu"],
     # attention over one latent row per token shared by all heads (keys and values per head are never formed), and the
     # per-head products around it
     "latent": ["attention_latent.cu", "attention_latent_mma.cu"],

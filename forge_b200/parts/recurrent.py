@@ -346,7 +346,8 @@ class GatedDeltaMixer(Part):
         rows = torch.cat([tensors[self._n(m)] for m in ("q", "k", "v", "g", "b", "a")], dim=0)
         pad = -rows.shape[0] % self.ROW_MULTIPLE
         self.proj = Linear(self._matrix(torch.cat([rows, rows.new_zeros(pad, rows.shape[1])], dim=0)), None, self.rt)
-        self.conv = self._vector_f32(torch.cat([tensors[self._n(m + ".conv")] for m in "qkv"], dim=0))
+        # [taps, channels], the current token's weights first: neighbouring threads read neighbouring channels
+        self.conv = self._vector_f32(torch.cat([tensors[self._n(m + ".conv")] for m in "qkv"], dim=0).flip(1).t())
         self.decay_rate = self._vector_f32(torch.exp(tensors[self._n("A_log")].to(torch.float64)))
         self.dt = self._vector_f32(tensors[self._n("dt_bias")])
         self.norm = self._vector_f32(tensors[self._n("norm")])
