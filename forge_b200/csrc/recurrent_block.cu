@@ -11,14 +11,14 @@
 // products k_i . k_j and k_i . q_j are the same for all columns and heads that share q and k: gram_kernel makes them ahead.  Every R is
 // the product of its decays (no quotients), so a decay of zero does no harm.
 //
-// A CTA of 64 threads has 16 columns of one head's S and walks a request's tokens of the step; eight threads share two columns, thread q of
+// A CTA has 16 columns of one head's S and walks a request's tokens of the step; eight threads share two columns (or one), thread q of
 // them holds the rows (4m + e) with m % 8 == q, as pairs of rows that one instruction multiplies and adds (fma.rn.f32x2).  The next
-// block's vectors are copied into the other half of the staging buffers (cp.async) while the present one is worked on.
+// blocks' vectors are copied into a ring of staging buffers (cp.async) while the present one is worked on.
 #include "common.cuh"
 
 namespace {
 
-constexpr int BT = 8, kCols = 16, kThreads = 64, kOStride = 12;
+constexpr int BT = 8, kCols = 16, kGramThreads = 64, kOStride = 12;
 typedef unsigned long long u64;
 
 __device__ __forceinline__ u64 fma2(u64 a, u64 b, u64 c) {
@@ -53,7 +53,7 @@ __device__ __forceinline__ int first_block(const int32_t* __restrict__ q_start, 
 
 // gram[block][head of q and k][a][b]: k_a . q_b for a <= b, k_a . k_b for a > b.  One CTA per (block, head); rows of zeros for the tokens
 // that a request's last block does not have.
-__global__ void __launch_bounds__(kThreads)
+__global__ void __launch_bounds__(kGramThreads)
 gram_kernel(const float* __restrict__ q, int ld_q, const float* __restrict__ k, int ld_k, const int32_t* __restrict__ q_start, int S, int M, int K,
             int stride, float* __restrict__ gram) {
     extern __shared__ __align__(16) float sm[];          // [k_0 .. k_7 | q_0 .. q_7], rows of `stride` numbers
@@ -68,7 +68,7 @@ gram_kernel(const float* __restrict__ q, int ld_q, const float* __restrict__ k, 
     const int t0 = q_start[lo] + (block - first_block(q_start, lo)) * BT, n = min(BT, q_start[lo + 1] - t0);
     if (n <= 0) return;
     for (int row = 0; row < BT; ++row)
-        for (int c = tid; c < stride; c += kThreads) {
+        for (int c = tid; c < stride; c += kGramThreads) {
             const bool ok = row < n && c < K;
             sm[row * stride + c] = ok ? k[(size_t)(t0 + row) * ld_k + head * K + c] : 0.f;
             sm[(BT + row) * stride + c] = ok ? q[(size_t)(t0 + row) * ld_q + head * K + c] : 0.f;
@@ -101,28 +101,30 @@ struct BlockScan {
     int N, M, K, KV, vec;
 };
 
-template <int KMAX, bool DELTA>
-__global__ void __launch_bounds__(kThreads)
+template <int KMAX, int CT, bool DELTA>
+__global__ void __launch_bounds__(8 * kCols / CT)
 block_scan_kernel(const BlockScan d) {
+    constexpr int kThreads = 8 * kCols / CT;              // CT: columns of S per thread
     constexpr int C4 = KMAX / 32, LD = KMAX + 4;          // float4 pieces of a column per thread; row length of the staged vectors
-    constexpr bool kHoldK = KMAX <= 64;                   // the keys stay in registers from the looks at S to its update
-    __shared__ __align__(16) float ks[2][BT][LD], qs[2][BT][LD], vs[2][BT][kCols], gs[2][BT], bs[2][BT], grams[2][BT * BT];
+    constexpr bool kHoldK = KMAX <= 64;                  // the keys stay in registers from the looks at S to its update
+    constexpr int kStages = KMAX > 64 && KMAX <= 128 ? 4 : 2;      // blocks on their way (heads of 128: 514 us with two, 424 with four)
+    __shared__ __align__(16) float ks[kStages][BT][LD], qs[kStages][BT][LD], vs[kStages][BT][kCols], gs[kStages][BT], bs[kStages][BT], grams[kStages][BT * BT];
     __shared__ __align__(16) float om[BT * kOStride], mm[BT * BT];
     forge::pdl_launch_dependents();
     const int s = blockIdx.x, head = blockIdx.y, tid = threadIdx.x, q = tid & 7, jp = tid >> 3;
     const int K = d.K, KV = d.KV, N = d.N, hk = head / (N / d.M);
-    const int col0 = blockIdx.z * kCols, j0 = col0 + 2 * jp;
+    const int col0 = blockIdx.z * kCols, j0 = col0 + CT * jp;
     // channels beyond K stay zero: the copies never touch them
-    for (int i = tid; i < 2 * BT * LD; i += kThreads) { (&ks[0][0][0])[i] = 0.f; (&qs[0][0][0])[i] = 0.f; }
+    for (int i = tid; i < kStages * BT * LD; i += kThreads) { (&ks[0][0][0])[i] = 0.f; (&qs[0][0][0])[i] = 0.f; }
     __syncthreads();
     forge::pdl_wait();
     const int t_lo = d.q_start[s], t_hi = d.q_start[s + 1];
     if (t_lo >= t_hi) return;
     float* S_g = d.state + (size_t)d.slots[s] * d.stride + (size_t)head * K * KV;
     auto row_of = [&](int ii) { return ((ii >> 2) * 8 + q) * 4 + (ii & 3); };
-    u64 S2[2][C4 * 2];
+    u64 S2[CT][C4 * 2];
 #pragma unroll
-    for (int c = 0; c < 2; ++c)
+    for (int c = 0; c < CT; ++c)
 #pragma unroll
         for (int ii = 0; ii < C4 * 4; ii += 2) {
             const bool ok = j0 + c < KV;
@@ -158,13 +160,18 @@ block_scan_kernel(const BlockScan d) {
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    fetch(0, t_lo);
+#pragma unroll
+    for (int i = 0; i < kStages - 1; ++i) {
+        if (t_lo + i * BT < t_hi) fetch(i, t_lo + i * BT);
+        else asm volatile("cp.async.commit_group;" ::: "memory");
+    }
     int buf = 0;
-    for (int tb = t_lo; tb < t_hi; tb += BT, buf ^= 1) {
+    for (int tb = t_lo; tb < t_hi; tb += BT, buf = buf + 1 < kStages ? buf + 1 : 0) {
         const int n = min(BT, t_hi - tb);
-        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        asm volatile("cp.async.wait_group %0;" ::"n"(kStages - 2) : "memory");
         __syncthreads();                                  // the block has landed for every thread, and the one before is done with
-        if (tb + BT < t_hi) fetch(buf ^ 1, tb + BT);
+        if (tb + (kStages - 1) * BT < t_hi) fetch(buf > 0 ? buf - 1 : kStages - 1, tb + (kStages - 1) * BT);
+        else asm volatile("cp.async.commit_group;" ::: "memory");
         float g[BT];
         if (DELTA) {
             *reinterpret_cast<float4*>(&g[0]) = *reinterpret_cast<const float4*>(&gs[buf][0]);
@@ -174,7 +181,7 @@ block_scan_kernel(const BlockScan d) {
             for (int l = 0; l < BT; ++l) g[l] = l < n ? fixed : 1.0f;
         }
         // the triangles with their decays: thread (a, b) = (tid / 8, tid % 8) does entry (a, b)
-        {
+        if (kThreads == BT * BT || tid < BT * BT) {
             const int a = tid >> 3, b = tid & 7, lo = min(a, b), hi = max(a, b);
             float r = grams[buf][tid];
 #pragma unroll
@@ -183,7 +190,7 @@ block_scan_kernel(const BlockScan d) {
             if (DELTA && a > b) mm[a * BT + b] = r;       // token a's write takes R_ba (k_b . k_a) u_b
         }
         // the looks at S: partial sums of S^T k_t and S^T q_t over this thread's rows, pairs of rows side by side
-        u64 A[DELTA ? BT : 1][2], B[BT][2], kh[kHoldK ? BT : 1][C4 * 2];
+        u64 A[DELTA ? BT : 1][CT], B[BT][CT], kh[kHoldK ? BT : 1][C4 * 2];
 #pragma unroll
         for (int tt = 0; tt < BT; ++tt) {
             const ulonglong2* k4 = reinterpret_cast<const ulonglong2*>(&ks[buf][tt][0]) + q;
@@ -195,7 +202,7 @@ block_scan_kernel(const BlockScan d) {
                 if (DELTA || kHoldK) kk = k4[c4 * 8];
                 if (kHoldK) { kh[kHoldK ? tt : 0][2 * c4] = kk.x; kh[kHoldK ? tt : 0][2 * c4 + 1] = kk.y; }
 #pragma unroll
-                for (int c = 0; c < 2; ++c) {
+                for (int c = 0; c < CT; ++c) {
                     B[tt][c] = c4 == 0 ? mul2(S2[c][0], qq.x) : fma2(S2[c][2 * c4], qq.x, B[tt][c]);
                     B[tt][c] = fma2(S2[c][2 * c4 + 1], qq.y, B[tt][c]);
                     if (DELTA) {
@@ -207,9 +214,9 @@ block_scan_kernel(const BlockScan d) {
             }
         }
         // the eight threads' sums meet so that thread q ends with token q's
-        float a1[2], b1[2];
+        float a1[CT], b1[CT];
 #pragma unroll
-        for (int c = 0; c < 2; ++c) {
+        for (int c = 0; c < CT; ++c) {
             float x[BT], y[BT];
 #pragma unroll
             for (int tt = 0; tt < BT; ++tt) {
@@ -241,16 +248,15 @@ block_scan_kernel(const BlockScan d) {
         for (int l = 0; l < BT; ++l) p_q *= l <= q ? g[l] : 1.0f;
         __syncthreads();                                  // the triangles stand
         // the writes u of both columns, all eight tokens, in every thread
-        float u[BT][2];
+        float u[BT][CT];
         if (DELTA) {
-            float mine[2];
-            const float2 vq = *reinterpret_cast<const float2*>(&vs[buf][q][2 * jp]);
-            mine[0] = fmaf(-p_q, a1[0], vq.x);
-            mine[1] = fmaf(-p_q, a1[1], vq.y);
+            float mine[CT];
+#pragma unroll
+            for (int c = 0; c < CT; ++c) mine[c] = fmaf(-p_q, a1[c], vs[buf][q][CT * jp + c]);
 #pragma unroll
             for (int j = 0; j < BT; ++j) {
 #pragma unroll
-                for (int c = 0; c < 2; ++c) u[j][c] = __shfl_sync(0xffffffffu, mine[c], j, 8);
+                for (int c = 0; c < CT; ++c) u[j][c] = __shfl_sync(0xffffffffu, mine[c], j, 8);
             }
             float bt[BT];
             *reinterpret_cast<float4*>(&bt[0]) = *reinterpret_cast<const float4*>(&bs[buf][0]);
@@ -261,7 +267,7 @@ block_scan_kernel(const BlockScan d) {
                 *reinterpret_cast<float4*>(&m[0]) = *reinterpret_cast<const float4*>(&mm[j * BT]);
                 if (j > 4) *reinterpret_cast<float4*>(&m[4]) = *reinterpret_cast<const float4*>(&mm[j * BT + 4]);
 #pragma unroll
-                for (int c = 0; c < 2; ++c) {
+                for (int c = 0; c < CT; ++c) {
 #pragma unroll
                     for (int i = 0; i < j; ++i) u[j][c] = fmaf(-m[i], u[i][c], u[j][c]);
                     u[j][c] *= bt[j];
@@ -270,9 +276,8 @@ block_scan_kernel(const BlockScan d) {
         } else {
 #pragma unroll
             for (int j = 0; j < BT; ++j) {
-                const float2 vj = *reinterpret_cast<const float2*>(&vs[buf][j][2 * jp]);
-                u[j][0] = vj.x;
-                u[j][1] = vj.y;
+#pragma unroll
+                for (int c = 0; c < CT; ++c) u[j][c] = vs[buf][j][CT * jp + c];
             }
         }
         // token q's output
@@ -281,7 +286,7 @@ block_scan_kernel(const BlockScan d) {
             *reinterpret_cast<float4*>(&om8[0]) = *reinterpret_cast<const float4*>(&om[q * kOStride]);
             *reinterpret_cast<float4*>(&om8[4]) = *reinterpret_cast<const float4*>(&om[q * kOStride + 4]);
 #pragma unroll
-            for (int c = 0; c < 2; ++c) {
+            for (int c = 0; c < CT; ++c) {
                 float o = p_q * b1[c];
 #pragma unroll
                 for (int i = 0; i < BT; ++i) o = fmaf(om8[i], u[i][c], o);
@@ -290,16 +295,16 @@ block_scan_kernel(const BlockScan d) {
         }
         // the state after the block
         float w = 1.f;
-        u64 uw[BT][2];
+        u64 uw[BT][CT];
 #pragma unroll
         for (int i = BT - 1; i >= 0; --i) {
 #pragma unroll
-            for (int c = 0; c < 2; ++c) uw[i][c] = pack2(w * u[i][c], w * u[i][c]);
+            for (int c = 0; c < CT; ++c) uw[i][c] = pack2(w * u[i][c], w * u[i][c]);
             w *= g[i];
         }
         const u64 w2 = pack2(w, w);
 #pragma unroll
-        for (int c = 0; c < 2; ++c)
+        for (int c = 0; c < CT; ++c)
 #pragma unroll
             for (int ii = 0; ii < C4 * 2; ++ii) S2[c][ii] = mul2(S2[c][ii], w2);
 #pragma unroll
@@ -311,7 +316,7 @@ block_scan_kernel(const BlockScan d) {
                 if (kHoldK) { kk.x = kh[kHoldK ? tt : 0][2 * c4]; kk.y = kh[kHoldK ? tt : 0][2 * c4 + 1]; }
                 else kk = k4[c4 * 8];
 #pragma unroll
-                for (int c = 0; c < 2; ++c) {
+                for (int c = 0; c < CT; ++c) {
                     S2[c][2 * c4] = fma2(kk.x, uw[tt][c], S2[c][2 * c4]);
                     S2[c][2 * c4 + 1] = fma2(kk.y, uw[tt][c], S2[c][2 * c4 + 1]);
                 }
@@ -319,7 +324,7 @@ block_scan_kernel(const BlockScan d) {
         }
     }
 #pragma unroll
-    for (int c = 0; c < 2; ++c)
+    for (int c = 0; c < CT; ++c)
 #pragma unroll
         for (int ii = 0; ii < C4 * 4; ii += 2) {
             const float2 p = unpack2(S2[c][ii / 2]);
@@ -331,7 +336,7 @@ block_scan_kernel(const BlockScan d) {
 template <bool DELTA>
 int run(BlockScan d, float* gram, int T, int S, cudaStream_t stream) {
     const int stride = (d.K + 3) / 4 * 4 + 4, blocks = T / BT + S;
-    cudaError_t e = forge::launch(gram_kernel, dim3(blocks, d.M), dim3(kThreads), sizeof(float) * 2 * BT * stride, stream, 1, d.q, d.ld_q, d.k, d.ld_k,
+    cudaError_t e = forge::launch(gram_kernel, dim3(blocks, d.M), dim3(kGramThreads), sizeof(float) * 2 * BT * stride, stream, 1, d.q, d.ld_q, d.k, d.ld_k,
                                   d.q_start, S, d.M, d.K, stride, gram);
     if (e != cudaSuccess) return forge::check_launch("block_scan (products)", e);
     auto aligned = [](const float* p, int ld) { return ((uintptr_t)p & 15) == 0 && ld % 4 == 0; };
@@ -339,9 +344,15 @@ int run(BlockScan d, float* gram, int T, int S, cudaStream_t stream) {
     d.vec = d.K % 4 == 0 && aligned(d.q, d.ld_q) && aligned(d.k, d.ld_k) ? 1 : 0;
     const dim3 grid(S, d.N, (d.KV + kCols - 1) / kCols);
     const int kmax = (d.K + 31) / 32 * 32;
-#define FORGE_BLOCK_CASE(KM) \
-    if (kmax <= KM) return forge::check_launch("block_scan", forge::launch(block_scan_kernel<KM, DELTA>, grid, dim3(kThreads), 0, stream, 1, d));
-    FORGE_BLOCK_CASE(32) FORGE_BLOCK_CASE(64) FORGE_BLOCK_CASE(96) FORGE_BLOCK_CASE(128) FORGE_BLOCK_CASE(192) FORGE_BLOCK_CASE(256)
+    // a column per thread where the CTAs do not even fill the SMs (one request, 32 heads of 64 x 64: 245 us for 2,048 tokens, with two
+    // columns 290), else two (64 heads: 304 us, with one column 336)
+    const bool few = (long long)S * d.N * grid.z <= 148;
+#define FORGE_BLOCK_CASE(KM, CT) \
+    if (kmax <= KM) return forge::check_launch("block_scan", forge::launch(block_scan_kernel<KM, CT, DELTA>, grid, dim3(8 * kCols / CT), 0, stream, 1, d));
+    if (few) {
+        FORGE_BLOCK_CASE(32, 1) FORGE_BLOCK_CASE(64, 1)
+    }
+    FORGE_BLOCK_CASE(32, 2) FORGE_BLOCK_CASE(64, 2) FORGE_BLOCK_CASE(96, 2) FORGE_BLOCK_CASE(128, 2) FORGE_BLOCK_CASE(192, 2) FORGE_BLOCK_CASE(256, 2)
 #undef FORGE_BLOCK_CASE
     return forge::fail(FORGE_ERR_UNSUPPORTED, "block_scan: heads of %d key channels (at most 256)", d.K);
 }

@@ -21,7 +21,8 @@ struct Columns {                      // a [T, n] fp32 matrix that may be a colu
 };
 
 __device__ __forceinline__ float sigmoidf(float x) { return 1.0f / (1.0f + expf(-x)); }
-__device__ __forceinline__ float siluf(float x) { return x * sigmoidf(x); }
+// (a denominator beyond 2^126 gives the 0 that the quotient would round to, or all but)
+__device__ __forceinline__ float siluf(float x) { return __fdividef(x, 1.0f + expf(-x)); }
 __device__ __forceinline__ float softplusf(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
 // exp(-x) of a small x is a number just below one that hundreds of tokens multiply: 1 + (exp(-x) - 1) is it to the last bit, where an
@@ -34,10 +35,11 @@ struct ShortConv {
     int channels;                     // numbers in a row of the ring (all tensors that are convolved, side by side)
 };
 
-constexpr int kTaps = 8;              // taps whose inputs and weights are all asked for before the first is used
+// TP (4 or 8, the kernels' template parameter): taps whose inputs and weights are all asked for before the first is used.
 
 // The convolution of channel c (its column of w and its place in the ring) of token t at position pos; x: the channel's numbers in the
 // projection; `first`: the request's first token of the step; ring: the request's ring.  The oldest input is added first, whatever the cut.
+template <int TP>
 __device__ __forceinline__ float convolve(const ShortConv& cv, const float* __restrict__ x, int ld, int t, int first, int pos, int c,
                                           const float* __restrict__ ring) {
     const int at = pos % cv.taps;
@@ -46,11 +48,11 @@ __device__ __forceinline__ float convolve(const ShortConv& cv, const float* __re
         return ring[(size_t)(at >= j ? at - j : at - j + cv.taps) * cv.channels + c];
     };
     float a = 0.f;
-    for (int j = cv.taps - 1; j >= kTaps; --j)
+    for (int j = cv.taps - 1; j >= TP; --j)
         if (pos >= j) a = fmaf(cv.w[(size_t)j * cv.channels + c], input(j), a);
-    float v[kTaps], w[kTaps];
+    float v[TP], w[TP];
 #pragma unroll
-    for (int j = 0; j < kTaps; ++j) {
+    for (int j = 0; j < TP; ++j) {
         v[j] = w[j] = 0.f;
         if (j < cv.taps && pos >= j) {
             v[j] = input(j);
@@ -58,7 +60,7 @@ __device__ __forceinline__ float convolve(const ShortConv& cv, const float* __re
         }
     }
 #pragma unroll
-    for (int j = kTaps - 1; j >= 0; --j) a = fmaf(w[j], v[j], a);
+    for (int j = TP - 1; j >= 0; --j) a = fmaf(w[j], v[j], a);
     return a;
 }
 
@@ -78,25 +80,25 @@ struct DeltaPrepare {
 
 constexpr int kUnitRegs = 8;          // channels of a q or k head that a lane holds (heads of up to 256)
 constexpr int kPrepTokens = 4;        // consecutive tokens that a warp takes at a time, so that most inputs are read once
-constexpr int kPrepTiles = 4;         // such tiles that a warp takes one after the other
 
 // kPrepTokens neighbouring tokens of one channel, t0 the first.  inner: all of them and all that they look back on are one request's
-// tokens of this step (and n == kPrepTokens, taps <= kTaps); then a window of inputs is read once and slides over the taps.
+// tokens of this step (and n == kPrepTokens, taps <= TP); then a window of inputs is read once and slides over the taps.
+template <int TP>
 __device__ __forceinline__ void convolve_tile(const DeltaPrepare& d, const float* __restrict__ x, int c, int t0, int n, bool inner, float (&y)[kPrepTokens]) {
     if (inner) {
-        float v[kTaps - 1 + kPrepTokens], w[kTaps];
+        float v[TP - 1 + kPrepTokens], w[TP];
 #pragma unroll
-        for (int i = 0; i < kTaps - 1 + kPrepTokens; ++i) {               // v[i]: token t0 + i - (kTaps - 1)
-            const int back = kTaps - 1 - i;
-            v[i] = back < d.cv.taps ? x[(ptrdiff_t)(t0 - back) * d.p.ld] : 0.f;
+        for (int i = 0; i < TP - 1 + kPrepTokens; ++i) {               // v[i]: token t0 + i - (TP - 1)
+            const int back = TP - 1 - i;
+            v[i] = back < d.cv.taps ? __ldg(x + (ptrdiff_t)(t0 - back) * d.p.ld) : 0.f;
         }
 #pragma unroll
-        for (int j = 0; j < kTaps; ++j) w[j] = j < d.cv.taps ? d.cv.w[(size_t)j * d.cv.channels + c] : 0.f;
+        for (int j = 0; j < TP; ++j) w[j] = j < d.cv.taps ? __ldg(d.cv.w + (size_t)j * d.cv.channels + c) : 0.f;
 #pragma unroll
         for (int k = 0; k < kPrepTokens; ++k) {
             float a = 0.f;
 #pragma unroll
-            for (int j = kTaps - 1; j >= 0; --j) a = fmaf(w[j], v[kTaps - 1 + k - j], a);
+            for (int j = TP - 1; j >= 0; --j) a = fmaf(w[j], v[TP - 1 + k - j], a);
             y[k] = siluf(a);
         }
         return;
@@ -105,12 +107,12 @@ __device__ __forceinline__ void convolve_tile(const DeltaPrepare& d, const float
         y[k] = 0.f;
         if (k >= n) continue;
         const int t = t0 + k, s = d.tok_req[t];
-        y[k] = siluf(convolve(d.cv, x, d.p.ld, t, d.q_start[s], d.positions[t], c, d.state + (size_t)d.slots[s] * d.stride + d.ring_off));
+        y[k] = siluf(convolve<TP>(d.cv, x, d.p.ld, t, d.q_start[s], d.positions[t], c, d.state + (size_t)d.slots[s] * d.stride + d.ring_off));
     }
 }
 
 // One tile of one head of q, k or v, by a warp.  NC: the lanes' channels of a q or k head.
-template <int NC>
+template <int NC, int TP>
 __device__ __forceinline__ void prepare_tile(const DeltaPrepare& d, int t0, int n, bool inner, int unit, int lane) {
     const int C = 2 * d.M * d.K + d.N * d.V;
     if (unit < 2 * d.M) {
@@ -122,7 +124,7 @@ __device__ __forceinline__ void prepare_tile(const DeltaPrepare& d, int t0, int 
         for (int i = 0; i < NC; ++i) {
             const int c = lane + 32 * i;
             if (32 * i >= d.K) continue;                                  // (the same for the whole warp)
-            if (c < d.K) convolve_tile(d, d.p.p + c0 + c, c0 + c, t0, n, inner, x[i]);
+            if (c < d.K) convolve_tile<TP>(d, d.p.p + c0 + c, c0 + c, t0, n, inner, x[i]);
 #pragma unroll
             for (int k = 0; k < kPrepTokens; ++k) {
                 if (c >= d.K) x[i][k] = 0.f;
@@ -145,7 +147,7 @@ __device__ __forceinline__ void prepare_tile(const DeltaPrepare& d, int t0, int 
     const int head = unit - 2 * d.M, c0 = 2 * d.M * d.K + head * d.V;
     for (int c = lane; c < d.V; c += 32) {
         float y[kPrepTokens];
-        convolve_tile(d, d.p.p + c0 + c, c0 + c, t0, n, inner, y);
+        convolve_tile<TP>(d, d.p.p + c0 + c, c0 + c, t0, n, inner, y);
 #pragma unroll
         for (int k = 0; k < kPrepTokens; ++k)
             if (k < n) d.qkv[(size_t)(t0 + k) * C + c0 + c] = y[k];
@@ -157,24 +159,24 @@ __device__ __forceinline__ void prepare_tile(const DeltaPrepare& d, int t0, int 
     }
 }
 
-// A warp per (kPrepTiles tiles of kPrepTokens tokens, head of q, k or v).
-template <int NC>
-__global__ void __launch_bounds__(128, NC <= 4 ? 6 : 4)
-delta_prepare_kernel(const DeltaPrepare d) {
+// A warp per (`tiles` tiles of kPrepTokens tokens, head of q, k or v).
+template <int NC, int TP>
+__global__ void __launch_bounds__(128, NC <= 4 ? 8 : 4)
+delta_prepare_kernel(const DeltaPrepare d, int tiles) {
     forge::pdl_wait();
-    const int first = (blockIdx.x * 4 + (threadIdx.x >> 5)) * kPrepTokens * kPrepTiles, lane = threadIdx.x & 31;
+    const int first = (blockIdx.x * 4 + (threadIdx.x >> 5)) * kPrepTokens * tiles, lane = threadIdx.x & 31;
     if (first >= d.T) return;
-    const int last = min(first + kPrepTokens * kPrepTiles, d.T) - 1, s0 = d.tok_req[first], back = d.cv.taps - 1;
-    const bool one = d.cv.taps <= kTaps && d.tok_req[last] == s0 && first - back >= d.q_start[s0];
+    const int last = min(first + kPrepTokens * tiles, d.T) - 1, s0 = d.tok_req[first], back = d.cv.taps - 1;
+    const bool one = d.cv.taps <= TP && d.tok_req[last] == s0 && first - back >= d.q_start[s0];
 #pragma unroll 1
     for (int t0 = first; t0 <= last; t0 += kPrepTokens) {
         const int n = min(kPrepTokens, d.T - t0);
         bool inner = one;
-        if (!one && d.cv.taps <= kTaps) {
+        if (!one && d.cv.taps <= TP) {
             const int s = d.tok_req[t0];
             inner = d.tok_req[t0 + n - 1] == s && t0 - back >= d.q_start[s];
         }
-        prepare_tile<NC>(d, t0, n, inner && n == kPrepTokens, blockIdx.y, lane);
+        prepare_tile<NC, TP>(d, t0, n, inner && n == kPrepTokens, blockIdx.y, lane);
     }
 }
 
@@ -278,7 +280,7 @@ struct TokenState {
 // added in a fixed order, and with u = beta (v - g S^T k) the output is g S^T q + (k . q) u.  Else S <- decay S + k v^T, o = S^T q.
 // out: DELTA: the normed and gated heads in the activation type; else the heads as they are, fp32.
 // kMost: the most threads of a launch, kCtas: how many such CTAs an SM should hold.
-template <int P, int kHeld, int kMost, int kCtas, bool DELTA, typename TA>
+template <int P, int kHeld, int kMost, int kCtas, int TP, bool DELTA, typename TA>
 __global__ void __launch_bounds__(kMost, kCtas)
 token_state_kernel(const TokenState d, TA* __restrict__ out, long long out_ld) {
     using S4 = typename Pack<P>::type;
@@ -321,11 +323,11 @@ token_state_kernel(const TokenState d, TA* __restrict__ out, long long out_ld) {
         for (int i = tid; i < 2 * K + V; i += threads) {
             // q and k of the shared head, then the head's values: column of the projection's [q | k | v] and of the ring
             const int c = i < K ? hk * K + i : (i < 2 * K ? (d.M - 1 + hk) * K + i : 2 * (d.M - 1) * K + head * V + i);
-            sm[i] = siluf(convolve(d.cv, d.q.p + c, d.q.ld, t, t, pos, c, ring));
+            sm[i] = siluf(convolve<TP>(d.cv, d.q.p + c, d.q.ld, t, t, pos, c, ring));
             // the token's own row of the ring, which nobody reads in this step
             if (i >= 2 * K || head % share == 0) now[c] = d.q.p[(size_t)t * d.q.ld + c];
         }
-        g = decayf(rate * softplusf(a_in));
+        g = decayf(rate * softplusf(a_in));                // (in every thread: one thread's would be waited for)
         beta = sigmoidf(b_in);
     } else {
         g = d.decay[head];
@@ -466,11 +468,11 @@ bool token_vec(const void* state, long long stride, int K, int V) {
     return V % 4 == 0 && K % 2 == 0 && stride % 4 == 0 && ((uintptr_t)state & 15) == 0;
 }
 
-template <bool DELTA, typename TO>
+template <int TP, bool DELTA, typename TO>
 cudaError_t launch_token(bool vec, const TokenShape& sh, dim3 grid, cudaStream_t stream, const TokenState& d, TO* out, long long out_ld) {
     const bool few = (d.K + sh.RG - 1) / sh.RG <= kHeld / 2;            // rows a thread holds: half the registers where half are enough
-    auto kernel = vec ? (few && sh.threads == 128 ? token_state_kernel<4, kHeld / 2, 128, 5, DELTA, TO> : token_state_kernel<4, kHeld, kTokenThreads, 1, DELTA, TO>)
-                      : (few ? token_state_kernel<1, kHeld / 2, kTokenThreads, 1, DELTA, TO> : token_state_kernel<1, kHeld, kTokenThreads, 1, DELTA, TO>);
+    auto kernel = vec ? (few && sh.threads == 128 ? token_state_kernel<4, kHeld / 2, 128, 6, TP, DELTA, TO> : token_state_kernel<4, kHeld, kTokenThreads, 1, TP, DELTA, TO>)
+                      : token_state_kernel<1, kHeld, kTokenThreads, 1, TP, DELTA, TO>;
     return forge::launch(kernel, grid, dim3(sh.threads), sh.smem, stream, 1, d, out, out_ld);
 }
 
@@ -492,9 +494,13 @@ extern "C" int forge_delta_prepare(const float* proj, int ld, int b_col, int a_c
     if (T == 0 || S == 0) return FORGE_OK;
     const ShortConv cv{conv_w, taps, (int)C};
     const DeltaPrepare d{{proj, ld}, b_col, a_col, cv, state, stride, ring_off, tok_req, q_start, positions, slots, decay_rate, dt, qkv, g, beta, T, N, M, K, V};
-    constexpr int per_cta = 4 * kPrepTokens * kPrepTiles;
-    cudaError_t e = forge::launch(K <= 64 ? delta_prepare_kernel<2> : K <= 128 ? delta_prepare_kernel<4> : delta_prepare_kernel<kUnitRegs>,
-                                  dim3((T + per_cta - 1) / per_cta, 2 * M + N), dim3(128), 0, stream, 1, d);
+    // several tiles one after the other in a warp as long as the SMs stay full
+    int tiles = 1;
+    while (tiles < 4 && (long long)(T / (4 * kPrepTokens * 2 * tiles)) * (2 * M + N) >= 148 * 8) tiles *= 2;
+    const int per_cta = 4 * kPrepTokens * tiles;
+    auto kernel = taps <= 4 ? (K <= 64 ? delta_prepare_kernel<2, 4> : K <= 128 ? delta_prepare_kernel<4, 4> : delta_prepare_kernel<kUnitRegs, 4>)
+                            : (K <= 64 ? delta_prepare_kernel<2, 8> : K <= 128 ? delta_prepare_kernel<4, 8> : delta_prepare_kernel<kUnitRegs, 8>);
+    cudaError_t e = forge::launch(kernel, dim3((T + per_cta - 1) / per_cta, 2 * M + N), dim3(128), 0, stream, 1, d, tiles);
     if (e != cudaSuccess) return forge::check_launch("delta_prepare", e);
     e = forge::launch(conv_keep_kernel, dim3(S, (unsigned)((C + 255) / 256)), dim3(256), 0, stream, 1, Columns{proj, ld}, cv, state, stride, ring_off,
                       q_start, positions, slots);
@@ -550,7 +556,7 @@ extern "C" int forge_gated_delta_token(const float* proj, int ld, int g_col, int
                        decay_rate, dt, state, stride, ring_off, q_start, positions, slots, weight, eps, N, M, K, V, sh.CG, sh.RG};
     cudaError_t e = cudaSuccess;
     FORGE_DISPATCH_DTYPE(dtype, TO,
-        e = launch_token<true>(vec, sh, dim3(S, N), stream, d, (TO*)out, out_ld));
+        e = taps <= 4 ? launch_token<4, true>(vec, sh, dim3(S, N), stream, d, (TO*)out, out_ld) : launch_token<8, true>(vec, sh, dim3(S, N), stream, d, (TO*)out, out_ld));
     return forge::check_launch("gated_delta_token", e);
 }
 
@@ -566,5 +572,5 @@ extern "C" int forge_lightning_token(const float* proj, int ld, const float* dec
     if (S == 0) return FORGE_OK;
     const TokenState d{{proj, ld}, {proj + N * K, ld}, {proj + 2 * N * K, ld}, {nullptr, 1, 0}, {nullptr, 0}, {nullptr, 0}, {nullptr, 0},
                        decay, nullptr, state, stride, 0, q_start, nullptr, slots, nullptr, 0.f, N, N, K, V, sh.CG, sh.RG};
-    return forge::check_launch("lightning_token", launch_token<false>(vec, sh, dim3(S, N), stream, d, out, (long long)N * V));
+    return forge::check_launch("lightning_token", launch_token<4, false>(vec, sh, dim3(S, N), stream, d, out, (long long)N * V));
 }

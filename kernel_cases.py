@@ -324,7 +324,44 @@ def case(name):
         batch = SimpleNamespace(q_start=i32(list(range(B + 1))), slots=i32(list(range(B))), num_requests=B, num_tokens=B)
         return (lambda: gla_token((qq, 0), (kk, 0), (v, 0), (g, 0), (u, 0), r, w2t, b, 16.0, batch, state, N, K, K, nw, 1e-5, torch.bfloat16)), \
             B * N * K * (2 * 4 * K + 4 * 4 + 2), 5 * B * N * K * K
-    raise SystemExit(f"unknown case {name!r}; known: depth_step_prefill depth_step_decode gla_scan gla_token_decode windowed_attention_prefill chunked_attention_prefill windowed_attention_decode windowed_latent_prefill windowed_latent_decode streams_mix_prefill streams_mix_decode routed_pairs_decode latent_attention_prefill latent_attention_prefill_512 latent_attention_decode retention_scan scored_attention_prefill scored_attention_decode distance_attention_prefill state_scan_gated headmix_attention_prefill headmix_attention_decode state_scan_wkv state_scan_delta "
+    if name in ("gated_delta_prepare", "gated_delta_scan", "gated_delta_token", "lightning_scan", "lightning_token"):
+        # the gated delta rule (32 heads of 64 x 64, two of which share a query/key head, convolutions over four tokens) and lightning
+        # attention (32 heads of 64 x 64): one request of 1,024 tokens, or single tokens of 256 requests (the state read and written
+        # once: 268 MB).  Algorithmic bytes of a portion: its inputs and outputs; FLOPs 6 (4) per state element and token
+        from forge_b200 import kernels as fk
+        N, M, K, taps = 32, 16, 64, 4
+        single = name.endswith("token")
+        B, T = (256, 256) if single else (1, 1024)
+        C = 2 * M * K + N * K
+        p, pl = torch.randn(T, C + N * K + 2 * N, device=DEV), torch.randn(T, 4 * N * K, device=DEV)
+        conv, rate, dt = torch.randn(taps, C, device=DEV) * 0.5, torch.rand(N, device=DEV) * 0.01, torch.zeros(N, device=DEV)
+        decay, nw = torch.full((N,), 0.99, device=DEV), torch.ones(K, device=DEV)
+        i32 = lambda z: torch.tensor(z, dtype=torch.int32, device=DEV)
+        pos = [100] * B if single else list(range(T))
+        batch = SimpleNamespace(q_start=i32(list(range(B + 1)) if single else [0, T]), slots=i32(list(range(B))), positions=i32(pos), num_requests=B,
+                                tok_req=i32(list(range(B)) if single else [0] * T), num_tokens=T)
+        state, lstate = torch.zeros(B, N * K * K + taps * C, device=DEV), torch.zeros(B, N * K * K, device=DEV)
+        cols = (0, C + N * K, C + N * K + N)
+        if name == "gated_delta_token":
+            return (lambda: fk.gated_delta_token(p, 0, C, *cols[1:], conv, rate, dt, batch, state, N, M, K, K, nw, 1e-5, torch.bfloat16)), \
+                B * (N * K * (2 * 4 * K + 4 + 2) + C * 4 * (taps + 1)), 6 * B * N * K * K
+        if name == "lightning_token":
+            return (lambda: fk.lightning_token(pl, 0, decay, batch, lstate, N, K, K)), B * N * K * (2 * 4 * K + 4 * 4), 4 * B * N * K * K
+        if name == "lightning_scan":
+            return (lambda: fk.lightning_scan(pl, 0, decay, batch, lstate, N, K, K)), 4 * T * N * K * 4, 4 * T * N * K * K
+        prepare = lambda: fk.gated_delta_prepare(p, *cols, conv, rate, dt, batch, state, N, M, K, K)
+        if name == "gated_delta_prepare":
+            return prepare, 2 * T * C * 4, 2 * T * C * taps
+        qkv, g, beta = prepare()
+        return (lambda: fk.gated_delta_scan(qkv, g, beta, batch, state, N, M, K, K)), T * (C + N * K) * 4, 6 * T * N * K * K
+    if name in ("join_prefill", "join_decode"):
+        # three outputs join a stream of 2,048 channels, two of them normed first, and the next layer's norm: 4,096 tokens (185 MB) or 8
+        from forge_b200.kernels import join
+        T, W_ = (4096 if name.endswith("prefill") else 8), 2048
+        x, ys, w = torch.randn(T, W_, device=DEV), [torch.randn(T, W_, device=DEV) for _ in range(3)], torch.ones(W_, device=DEV)
+        return (lambda: join(x, [(ys[0], w, 0.5), (ys[1], w, 0.5), (ys[2], None, 1.0)], 1e-5, next_norm=(w, 1e-5), out_dtype=torch.bfloat16)), \
+            T * W_ * (5 * 4 + 2), T * W_ * 14
+    raise SystemExit(f"unknown case {name!r}; known: gated_delta_prepare gated_delta_scan gated_delta_token lightning_scan lightning_token join_prefill join_decode depth_step_prefill depth_step_decode gla_scan gla_token_decode windowed_attention_prefill chunked_attention_prefill windowed_attention_decode windowed_latent_prefill windowed_latent_decode streams_mix_prefill streams_mix_decode routed_pairs_decode latent_attention_prefill latent_attention_prefill_512 latent_attention_decode retention_scan scored_attention_prefill scored_attention_decode distance_attention_prefill state_scan_gated headmix_attention_prefill headmix_attention_decode state_scan_wkv state_scan_delta "
                      "gemm_decode_gateup gemm_decode_down gemm_decode_lmhead gemm_prefill_qkv "
                      "gemm_prefill_gateup "
                      "gemm_prefill_qkv_rope gemm_prefill_down attention_decode attention_decode_fused attention_decode_stream attention_prefill "

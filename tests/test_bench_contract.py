@@ -129,3 +129,25 @@ def test_the_fifth_design_option_too():
     specs = Model(cfg.plan(), Runtime(torch.device("cpu"), torch.bfloat16)).tensor_specs()
     shapes = {n: s.default_shape or s.shape for n, s in specs.items() if s.required and n != "embed"}
     assert layers == sum(a[0] * a[1] for a in shapes.values() if len(a) == 2) and head == 300 * 256
+
+
+def test_the_sixth_design_option_too():
+    rc, lines = _run("--design", "zuretar", "--gpus", "2")
+    assert rc == 2 and len(lines) == 1 and "single-GPU" in json.loads(lines[0])["error"]
+    sys.path.insert(0, ROOT)
+    import bench
+    import torch
+    from forge_b200.config import config_from_dict
+    from forge_b200.engine.model import Model
+    from forge_b200.parts import Runtime
+    z = dict(width=256, layers=5, heads=8, kv_heads=2, dim=32, ff=512, state_heads=4, state_dim=32, rank=16, window=64, vocab=300)
+    cfg = config_from_dict(bench.zuretar_shape(**z))
+    assert [l["type"] for l in cfg.layers] == ["delta", "delta", "parallel", "delta", "delta"] and cfg.plan().schedule == [0, 1, 2, 0, 3]
+    # counted from the configuration alone with every expert read, the matrices are what the model's own tensor list holds, those of a
+    # layer that runs twice counted twice
+    layers, head = bench.zuretar_matmul_params(cfg, experts_read=8)
+    specs = Model(cfg.plan(), Runtime(torch.device("cpu"), torch.bfloat16)).tensor_specs()
+    sizes = {n: s.shape[0] * s.shape[1] for n, s in specs.items() if len(s.shape) == 2 and s.required and n not in ("embed", "head")}
+    assert layers == sum(sizes.values()) + sum(v for n, v in sizes.items() if n.startswith("l0.")) and head == 300 * 256
+    per_token, _ = bench.zuretar_matmul_params(cfg)
+    assert layers - per_token == 2 * 6 * 3 * 256 * 256                    # six of eight experts of two routed layers
